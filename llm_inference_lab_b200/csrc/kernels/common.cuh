@@ -98,9 +98,11 @@ __device__ __forceinline__ float lab_act(float z, int code) {
   return r * r;
 }
 
-// The gate of a gated pair of products, by its limit: 0, silu(g) * u; a positive limit, the capped form with
-// g' = min(g, limit) and u' = clamp(u, -limit, limit): g' * sigmoid(1.702 g') * (u' + 1).
-__device__ __forceinline__ float gate_pair(float g, float u, float limit) {
+// The gate of a gated pair of products.  `act` 1: the tanh form of GELU of g, times u; 0, by the limit: 0, silu(g) *
+// u; a positive limit, the capped form with g' = min(g, limit) and u' = clamp(u, -limit, limit): g' * sigmoid(1.702
+// g') * (u' + 1).
+__device__ __forceinline__ float gate_pair(float g, float u, int act, float limit) {
+  if (act == 1) return gelu_tanh_f(g) * u;
   if (limit > 0.f) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);

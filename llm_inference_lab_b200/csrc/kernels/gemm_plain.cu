@@ -20,7 +20,8 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(OutT* __restrict__ out,
                                                          int N, int K, int ldx, int ldo, long long batch_x,
                                                          long long batch_w, long long batch_o, int gelu,
                                                          const int* __restrict__ row_src, int row_div,
-                                                         const int* __restrict__ tile_group, float gate_limit) {
+                                                         const int* __restrict__ tile_group, int gate_act,
+                                                         float gate_limit, const float* __restrict__ row_scale) {
   pdl_trigger();
   pdl_wait();
   // a batch of products of one shape (blockIdx.z): operand b lies b * batch_* elements further on
@@ -84,14 +85,19 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(OutT* __restrict__ out,
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= M) continue;
+    float scale = 1.f;      // a gated row of the grouped layout may count as its scale times the row
+    if (GATED && row_scale != nullptr) {
+      const int src = row_src[m];
+      scale = src >= 0 ? row_scale[src] : 0.f;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       float v;
       if (GATED) {
-        const float g = acc[0][i][j], u = acc[GATED ? 1 : 0][i][j];
-        v = gate_pair(g, u, gate_limit);
+        const float g = acc[0][i][j] * scale, u = acc[GATED ? 1 : 0][i][j] * scale;
+        v = gate_pair(g, u, gate_act, gate_limit);
       } else {
         v = acc[0][i][j] + (bias ? to_f32<T>(bias[n]) : 0.f);
         if (gelu) v = lab_act(v, gelu);      // the activation after the bias, before the rounding
@@ -180,9 +186,11 @@ __global__ void __launch_bounds__(256) gemm_grouped_few_kernel(OutT* __restrict_
                                                                int ldo, long long group_w,
                                                                const int* __restrict__ row_src, int row_div,
                                                                int gather, const int* __restrict__ tile_group,
-                                                               int tile, int vec, float gate_limit) {
+                                                               int tile, int vec, int gate_act, float gate_limit,
+                                                               const float* __restrict__ row_scale) {
   __shared__ float xs[GF_ROWS][GF_KC];
   __shared__ int live_row[GF_TILE_MAX], live_x[GF_TILE_MAX];
+  __shared__ float live_scale[GF_TILE_MAX];      // gated: the row counts as its scale times the row
   __shared__ int n_live_s;
   pdl_trigger();
   pdl_wait();
@@ -206,6 +214,7 @@ __global__ void __launch_bounds__(256) gemm_grouped_few_kernel(OutT* __restrict_
     if (my_src >= 0) {
       live_row[at] = m0 + tid;
       live_x[at] = gather ? my_src / row_div : m0 + tid;
+      live_scale[at] = row_scale != nullptr ? row_scale[my_src] : 1.f;
     }
     if (tid == 0) n_live_s = all;
   }
@@ -282,9 +291,11 @@ __global__ void __launch_bounds__(256) gemm_grouped_few_kernel(OutT* __restrict_
       if (lane != 0) continue;
       OutT* dst = out + (size_t)live_row[r0 + t] * ldo;
       if (GATED) {
+        const float scale = live_scale[r0 + t];
 #pragma unroll
         for (int c = 0; c < NR / 2; ++c)
-          if (col[2 * c] < N) dst[col[2 * c]] = from_f32<OutT>(gate_pair(v[2 * c], v[2 * c + 1], gate_limit));
+          if (col[2 * c] < N)
+            dst[col[2 * c]] = from_f32<OutT>(gate_pair(v[2 * c] * scale, v[2 * c + 1] * scale, gate_act, gate_limit));
       } else {
 #pragma unroll
         for (int r = 0; r < NR; ++r)
@@ -297,7 +308,7 @@ __global__ void __launch_bounds__(256) gemm_grouped_few_kernel(OutT* __restrict_
 template <typename T, typename OutT>
 int launch_grouped_few(void* out, const void* x, const void* w, int M, int N, int K, int ldx, int ldo, int gated,
                        long long group_w, const int* row_src, int row_div, int gather, const int* tile_group, int tile,
-                       cudaStream_t stream, float gate_limit) {
+                       cudaStream_t stream, float gate_limit, const float* row_scale) {
   constexpr int V = 16 / (int)sizeof(T);
   const int vec = K % V == 0 && ((uintptr_t)w & 15) == 0;
   const int cols = gated ? 16 : 32;      // 8 warps, four weight rows each
@@ -305,28 +316,31 @@ int launch_grouped_few(void* out, const void* x, const void* w, int M, int N, in
   if (gated)
     return (int)lab_launch(gemm_grouped_few_kernel<T, OutT, true>, grid, dim3(256), 0, stream, (OutT*)out, (const T*)x,
                            (const T*)w, M, N, K, ldx, ldo, group_w, row_src, row_div, gather, tile_group, tile, vec,
-                           gate_limit);
+                           (int)(gated == 4), gate_limit, row_scale);
   return (int)lab_launch(gemm_grouped_few_kernel<T, OutT, false>, grid, dim3(256), 0, stream, (OutT*)out, (const T*)x,
-                         (const T*)w, M, N, K, ldx, ldo, group_w, row_src, row_div, gather, tile_group, tile, vec, 0.f);
+                         (const T*)w, M, N, K, ldx, ldo, group_w, row_src, row_div, gather, tile_group, tile, vec, 0,
+                         0.f, nullptr);
 }
 
 template <typename T, typename OutT>
 int launch(void* out, const void* x, const void* w, const void* bias, int M, int N, int K, int ldx, int ldo, int gated,
            cudaStream_t stream, int batch = 1, long long batch_x = 0, long long batch_w = 0, long long batch_o = 0,
-           const int* row_src = nullptr, int row_div = 1, const int* tile_group = nullptr, float gate_limit = 0.f) {
+           const int* row_src = nullptr, int row_div = 1, const int* tile_group = nullptr, float gate_limit = 0.f,
+           const float* row_scale = nullptr) {
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM, batch);
-  if (gated == 1)
+  if (gated == 1 || gated == 4)
     return (int)lab_launch(gemm_plain_kernel<T, OutT, true>, grid, dim3(256), 0, stream, (OutT*)out, (const T*)x,
                            (const T*)w, (const T*)nullptr, M, N, K, ldx, ldo, batch_x, batch_w, batch_o, 0, row_src,
-                           row_div, tile_group, gate_limit);
+                           row_div, tile_group, (int)(gated == 4), gate_limit, row_scale);
   return (int)lab_launch(gemm_plain_kernel<T, OutT, false>, grid, dim3(256), 0, stream, (OutT*)out, (const T*)x,
                          (const T*)w, (const T*)bias, M, N, K, ldx, ldo, batch_x, batch_w, batch_o,
-                         gated >= 2 ? gated - 1 : 0, row_src, row_div, tile_group, 0.f);
+                         gated >= 2 ? gated - 1 : 0, row_src, row_div, tile_group, 0, 0.f, nullptr);
 }
 }  // namespace
 
 // N is the number of output columns; with gated == 1, w holds 2 N rows (gate rows, then up rows); gated == 2 is
-// the plain product with GELU (tanh form) after the bias, 3 with the square of relu.
+// the plain product with GELU (tanh form) after the bias, 3 with the square of relu; 4 is the pair gated by the tanh
+// form of GELU (2 N rows as well).
 LAB_EXPORT int lab_gemm_plain(void* out, const void* x, const void* w, const void* bias, int M, int N, int K, int ldx,
                               int ldo, int gated, int dtype, int out_f32, float gate_limit, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
@@ -366,21 +380,23 @@ LAB_EXPORT int lab_gemm_plain_batched(void* out, const void* x, const void* w, i
 // matrix tile_group[t] of `w` (matrices group_w elements apart; -1: the tile holds no rows and is skipped); row m of
 // the product reads x's row row_src[m] / row_div (row_src null: row m itself; -1: padding, read as zeros).
 // M counts the rows of the grouped layout (out has that many); x must hold every row that row_src names.
+// row_scale (gated; null: none): the product of row m is that of row_scale[row_src[m]] times the row.
 LAB_EXPORT int lab_gemm_plain_group_rows() { return BM; }
 LAB_EXPORT int lab_gemm_plain_grouped(void* out, const void* x, const void* w, int M, int N, int K, int ldx, int ldo,
                                       int gated, long long group_w, const int* row_src, int row_div,
                                       const int* tile_group, int dtype, int out_f32, float gate_limit,
-                                      cudaStream_t stream) {
+                                      const float* row_scale, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (row_scale != nullptr && (!gated || row_src == nullptr)) return (int)cudaErrorInvalidValue;
   if (tile_group == nullptr || row_div < 1) return (int)cudaErrorInvalidValue;
   if (dtype == LAB_F32)
     return launch<float, float>(out, x, w, nullptr, M, N, K, ldx, ldo, gated, stream, 1, 0, group_w, 0, row_src, row_div,
-                                tile_group, gate_limit);
+                                tile_group, gate_limit, row_scale);
   if (out_f32)
     return launch<__nv_bfloat16, float>(out, x, w, nullptr, M, N, K, ldx, ldo, gated, stream, 1, 0, group_w, 0, row_src,
-                                        row_div, tile_group, gate_limit);
+                                        row_div, tile_group, gate_limit, row_scale);
   return launch<__nv_bfloat16, __nv_bfloat16>(out, x, w, nullptr, M, N, K, ldx, ldo, gated, stream, 1, 0, group_w, 0,
-                                              row_src, row_div, tile_group, gate_limit);
+                                              row_src, row_div, tile_group, gate_limit, row_scale);
 }
 
 // The same product for few rows (a decode step): tile t of `tile` rows (at most 128) meets matrix tile_group[t];
@@ -389,17 +405,18 @@ LAB_EXPORT int lab_gemm_plain_grouped(void* out, const void* x, const void* w, i
 LAB_EXPORT int lab_gemm_plain_grouped_few(void* out, const void* x, const void* w, int M, int N, int K, int ldx,
                                           int ldo, int gated, long long group_w, const int* row_src, int row_div,
                                           int gather, const int* tile_group, int tile, int dtype, int out_f32,
-                                          float gate_limit, cudaStream_t stream) {
+                                          float gate_limit, const float* row_scale, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (tile_group == nullptr || row_src == nullptr || row_div < 1 || tile < 1 || tile > GF_TILE_MAX || K <= 0)
     return (int)cudaErrorInvalidValue;
   if ((M + tile - 1) / tile > 65535) return (int)cudaErrorInvalidValue;
   if (dtype == LAB_F32)
     return launch_grouped_few<float, float>(out, x, w, M, N, K, ldx, ldo, gated, group_w, row_src, row_div, gather,
-                                            tile_group, tile, stream, gate_limit);
+                                            tile_group, tile, stream, gate_limit, row_scale);
   if (out_f32)
     return launch_grouped_few<__nv_bfloat16, float>(out, x, w, M, N, K, ldx, ldo, gated, group_w, row_src, row_div,
-                                                    gather, tile_group, tile, stream, gate_limit);
+                                                    gather, tile_group, tile, stream, gate_limit, row_scale);
   return launch_grouped_few<__nv_bfloat16, __nv_bfloat16>(out, x, w, M, N, K, ldx, ldo, gated, group_w, row_src,
-                                                          row_div, gather, tile_group, tile, stream, gate_limit);
+                                                          row_div, gather, tile_group, tile, stream, gate_limit,
+                                                          row_scale);
 }

@@ -107,7 +107,8 @@ struct Params {
   int k_tiles;          // k-tiles in total
   int k_tiles_per_split;
   int up_offset;        // gated: row offset of the "up" half inside the weight matrix
-  float gate_limit;     // gated: 0, silu(gate) * up; positive, the capped form (`silu_gate` with a limit)
+  int gate_act;         // gated: 0, by gate_limit; 1, the tanh form of GELU of the gate, times up
+  float gate_limit;     // gated: 0, silu(gate) * up; positive, the capped form (`gate_value` in tcgen05.cuh)
   int m_tiles, n_tiles, splits;  // tiles on the M side, on the N side, and split-K planes
   QkvStore qkv;         // q/k/v epilogue only
   PickArgs pick;        // picking head only
@@ -115,6 +116,10 @@ struct Params {
   // tile_group[t] * group_rows of the weight operand; a tile whose group is -1 holds no rows and is skipped.
   const int* tile_group;
   int group_rows;
+  // Gated grouped rows: with row_scale, gate and up of row m are multiplied by row_scale[row_src[m]] before the
+  // activation, as if the row itself had been (a row whose row_src is -1 holds nothing).
+  const float* row_scale;
+  const int* row_src;
 };
 
 // Element offset of (slot, kv head) in a cache of [pages, n_kv, page_size, d], or -1 (no slot; a
@@ -488,6 +493,13 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
         constexpr int OUT_COLS = GATED ? BN / 2 : BN;
         static_assert(OUT_COLS % 32 == 0, "normal orientation works on 32 output columns at a time");
         const int nbase = (n0 / N_ROWS) * OUT_COLS;
+        float scale = 1.f;
+        if constexpr (GATED) {
+          if (p.row_scale != nullptr && m < p.m_rows) {
+            const int src = p.row_src[m];
+            scale = src >= 0 ? p.row_scale[src] : 0.f;
+          }
+        }
 #pragma unroll 1
         for (int c = 0; c < OUT_COLS / 32 && go; ++c) {
           uint32_t r[32];
@@ -499,7 +511,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
               tmem_ld32_issue(lane_addr + BN / 2 + c * 32, ru);
               tmem_wait();
 #pragma unroll
-              for (int j = 0; j < 32; ++j) v[j] = silu_gate(__uint_as_float(r[j]), __uint_as_float(ru[j]), p.gate_limit);
+              for (int j = 0; j < 32; ++j)
+                v[j] = gate_value(__uint_as_float(r[j]) * scale, __uint_as_float(ru[j]) * scale, p.gate_act, p.gate_limit);
             } else {
               tmem_wait();
 #pragma unroll
@@ -597,7 +610,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
             const int tok = n0 + col;
             if (tok >= p.n_rows) break;
             dst[(size_t)tok * p.ld_out] =
-                __float2bfloat16_rn(silu_gate(exchange[f * (BN + 1) + col], exchange[(HALF + f) * (BN + 1) + col], p.gate_limit));
+                __float2bfloat16_rn(gate_value(exchange[f * (BN + 1) + col], exchange[(HALF + f) * (BN + 1) + col],
+                                               p.gate_act, p.gate_limit));
           }
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");  // the buffer is free for the next tile
@@ -782,14 +796,16 @@ __global__ void wait_probe_kernel(unsigned long long limit_ns, int* gave_up) {
 // out: bf16 or f32 [tokens, ld_out]; with splits > 1, `out` is the partial buffer
 // [splits, tokens, ld_out] of floats (no bias, not gated).
 // swap != 0: features on the M side (few tokens); bn: tile of the N side (16..256).
-// gated: 0 the plain product, 1 the SiLU-gated pair, 2 the plain product with GELU (tanh form) after the bias, 3 with the square of relu.
+// gated: 0 the plain product, 1 the SiLU-gated pair, 2 the plain product with GELU (tanh form) after the bias, 3 with the square of relu,
+// 4 the pair gated by the tanh form of GELU.
 // gate_limit (gated 1): 0, silu(gate) * up; positive, gate and up capped at the limit, sigmoid(1.702 gate), up + 1.
 LAB_EXPORT int lab_gemm_tc(void* out, const void* x, const void* w, const void* bias, int tokens, int n_out, int K,
                            int ldx, int ld_out, int gated, int out_f32, int swap, int bn, int splits,
                            float gate_limit, cudaStream_t stream) {
   if (tokens <= 0 || n_out <= 0) return 0;
-  const int gelu = gated >= 2 ? gated - 1 : 0;      // 1: GELU, 2: the square of relu
-  if (gelu) gated = 0;
+  const int gelu = gated == 2 || gated == 3 ? gated - 1 : 0;      // 1: GELU, 2: the square of relu
+  const int gate_act = gated == 4;
+  gated = gated == 1 || gated == 4;
   if (gelu && splits > 1) return (int)cudaErrorInvalidValue;
   if (K % 8 || ldx % 8 || K <= 0) return (int)cudaErrorInvalidValue;            // 16-byte rows for TMA
   if ((((uintptr_t)x) | ((uintptr_t)w)) & 15) return (int)cudaErrorInvalidValue;  // 16-byte bases for TMA
@@ -799,6 +815,7 @@ LAB_EXPORT int lab_gemm_tc(void* out, const void* x, const void* w, const void* 
   p.out = out;
   p.bias = (const __nv_bfloat16*)bias;
   p.gelu = gelu;
+  p.gate_act = gate_act;
   p.gate_limit = gate_limit;
   p.ld_out = ld_out;
   p.split_stride = splits > 1 ? (long long)tokens * ld_out : 0;
@@ -824,11 +841,17 @@ LAB_EXPORT int lab_gemm_tc(void* out, const void* x, const void* w, const void* 
 // Rows grouped by the matrix they meet (routed experts), tokens on the M side: tile t of lab_gemm_tc_group_rows()
 // rows of x [rows, K] meets matrix tile_group[t] of w [groups, n_out (x2 when gated: gate rows, then up rows), K]
 // (-1: the tile holds no rows; it is skipped and its rows of `out` stay unwritten).  rows is a multiple of the
-// tile.  out: bf16 or f32 [rows, ld_out]; gated: silu(gate) * up, bf16 only.  bn: 64, 128 or 256.
+// tile.  out: bf16 or f32 [rows, ld_out]; gated: 1 silu(gate) * up (or the capped form), 4 the tanh form of GELU of
+// the gate times up, bf16 only.  bn: 64, 128 or 256.  row_scale (gated; null: none): the product of row m is that of
+// row_scale[row_src[m]] times the row.
 LAB_EXPORT int lab_gemm_tc_group_rows() { return BM; }
 LAB_EXPORT int lab_gemm_tc_grouped(void* out, const void* x, const void* w, int rows, int n_out, int K, int ldx,
                                    int ld_out, int gated, int out_f32, int bn, int groups, const int* tile_group,
-                                   float gate_limit, cudaStream_t stream) {
+                                   float gate_limit, const float* row_scale, const int* row_src,
+                                   cudaStream_t stream) {
+  if (row_scale != nullptr && (!gated || row_src == nullptr)) return (int)cudaErrorInvalidValue;
+  const int gate_act = gated == 4;
+  gated = gated != 0;
   if (rows <= 0 || n_out <= 0) return 0;
   if (rows % BM || groups <= 0 || tile_group == nullptr || (gated && out_f32)) return (int)cudaErrorInvalidValue;
   if (K % 8 || ldx % 8 || K <= 0) return (int)cudaErrorInvalidValue;            // 16-byte rows for TMA
@@ -843,7 +866,10 @@ LAB_EXPORT int lab_gemm_tc_grouped(void* out, const void* x, const void* w, int 
   const int rc = set_up(p, ma, mb, grid, x, w, rows, n_out, (int)w_rows, K, ldx, gated, 0, bn, 1);
   if (rc) return rc;
   p.tile_group = tile_group;
+  p.gate_act = gate_act;
   p.gate_limit = gate_limit;
+  p.row_scale = row_scale;
+  p.row_src = row_src;
   p.group_rows = gated ? 2 * n_out : n_out;
   if (gated) return dispatch_bn<GATED_SILU, false, __nv_bfloat16>(bn, ma, mb, p, grid, stream);
   if (out_f32) return dispatch_bn<PLAIN, false, float>(bn, ma, mb, p, grid, stream);

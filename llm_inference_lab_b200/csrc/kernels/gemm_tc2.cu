@@ -99,7 +99,8 @@ struct Params {
   int k_tiles;          // k-tiles in total
   int k_tiles_per_split;
   int up_offset;        // gated: row offset of the "up" half inside the weight matrix
-  float gate_limit;     // gated: 0, silu(gate) * up; positive, the capped form (`silu_gate` with a limit)
+  int gate_act;         // gated: 0, by gate_limit; 1, the tanh form of GELU of the gate, times up
+  float gate_limit;     // gated: 0, silu(gate) * up; positive, the capped form (`gate_value` in tcgen05.cuh)
   int m_tiles, n_tiles, splits;  // tiles of 256 tokens, tiles of output features, split-K planes
 };
 
@@ -262,7 +263,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc2_kernel(const __grid_constant
             tmem_ld32_issue(lane_addr + BN / 2 + c * 32, ru);
             tmem_wait();
 #pragma unroll
-            for (int j = 0; j < 32; ++j) v[j] = silu_gate(__uint_as_float(r[j]), __uint_as_float(ru[j]), p.gate_limit);
+            for (int j = 0; j < 32; ++j)
+              v[j] = gate_value(__uint_as_float(r[j]), __uint_as_float(ru[j]), p.gate_act, p.gate_limit);
           } else {
             tmem_wait();
 #pragma unroll
@@ -427,13 +429,15 @@ int pick_bn(int tokens, int n_out, bool gated, int splits) {
 // out: bf16 or f32 [tokens, ld_out]; with splits > 1, `out` is the partial buffer
 // [splits, tokens, ld_out] of floats (no bias, not gated).
 // bn: accumulator columns of a tile, 256, 224 or 192; 0: the width that fills the rounds of the pairs best.
-// gated: 0 the plain product, 1 the SiLU-gated pair, 2 the plain product with GELU (tanh form) after the bias, 3 with the square of relu.
+// gated: 0 the plain product, 1 the SiLU-gated pair, 2 the plain product with GELU (tanh form) after the bias, 3 with the square of relu,
+// 4 the pair gated by the tanh form of GELU.
 LAB_EXPORT int lab_gemm_tc2(void* out, const void* x, const void* w, const void* bias, int tokens, int n_out, int K,
                             int ldx, int ld_out, int gated, int out_f32, int splits, int bn, float gate_limit,
                             cudaStream_t stream) {
   if (tokens <= 0 || n_out <= 0) return 0;
-  const int gelu = gated >= 2 ? gated - 1 : 0;      // 1: GELU, 2: the square of relu
-  if (gelu) gated = 0;
+  const int gelu = gated == 2 || gated == 3 ? gated - 1 : 0;      // 1: GELU, 2: the square of relu
+  const int gate_act = gated == 4;
+  gated = gated == 1 || gated == 4;
   if (gelu && splits > 1) return (int)cudaErrorInvalidValue;
   if (K % 8 || ldx % 8 || K <= 0) return (int)cudaErrorInvalidValue;            // 16-byte rows for TMA
   if ((((uintptr_t)x) | ((uintptr_t)w)) & 15) return (int)cudaErrorInvalidValue;  // 16-byte bases for TMA
@@ -450,6 +454,7 @@ LAB_EXPORT int lab_gemm_tc2(void* out, const void* x, const void* w, const void*
   p.out = out;
   p.bias = (const __nv_bfloat16*)bias;
   p.gelu = gelu;
+  p.gate_act = gate_act;
   p.gate_limit = gate_limit;
   p.tokens = tokens;
   p.n_out = n_out;

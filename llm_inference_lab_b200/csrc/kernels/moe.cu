@@ -1,16 +1,19 @@
 // Routed feed-forward layers (a mixture of experts): the router's choice, the layout of the chosen
 // (token, expert) pairs in rows grouped by expert, and the weighted sum of the experts' results.
 //
-//   scores  s = softmax(z) over all experts, z the router's logits in 32-bit
+//   scores  s = softmax(z) over all experts, or sigmoid(z), z the router's logits in 32-bit
 //   choice  the `top` largest scores of a token (ties: the smaller index)
 //   weights the chosen scores over their sum (+ 1e-20), or (renorm 0) the chosen scores as they are
-//   out[t]  = sum over the chosen of weight * expert's result  (+ sigmoid(g_t) * shared expert's result)
+//   out[t]  = sum over the chosen of weight * expert's result  (+ sigmoid(g_t) * shared expert's result); the plain
+//             sum of the results where the weights have multiplied the experts' inputs
 //
 // The grouped matrix products between these kernels read rows through `row_src` and pick a tile's matrix
 // by `tile_group` (see the product kernels): pair (t, k) lies at row pos_of[t * top + k] of the grouped
 // layout, every expert's rows start on a tile border, unused rows are marked -1.  Where a pair lands inside
 // its expert's rows depends on timing; no result does: the sum over a token's experts runs in the order of
 // its choice.
+#include <cfloat>
+
 #include "common.cuh"
 
 namespace {
@@ -18,52 +21,55 @@ constexpr int kThreads = 256;
 constexpr int kWarps = kThreads / 32;
 
 // One warp per token.  logits [tokens, ld]: the experts' logits at columns [0, E); column `gate_col` (if
-// >= 0) holds the logit of the shared expert's gate.
+// >= 0) holds the logit of the shared expert's gate.  Both kinds of score grow with the logit, so the choice
+// compares logits.
 __global__ void __launch_bounds__(kThreads) moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight,
                                                              float* __restrict__ shared_gate,
                                                              const float* __restrict__ logits, int ld, int tokens,
-                                                             int E, int top, int gate_col, int renorm) {
-  extern __shared__ float scores[];      // [kWarps][E]
+                                                             int E, int top, int gate_col, int renorm, int sigmoid) {
+  extern __shared__ float keys[];      // [kWarps][E]
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kWarps + warp;
   if (t >= tokens) return;
-  float* s = scores + (size_t)warp * E;
+  float* s = keys + (size_t)warp * E;
   const float* z = logits + (size_t)t * ld;
+  // A logit that is no number (a row of padding may hold anything) counts as the smallest number, and a taken
+  // expert as less than any, so that every choice names an expert that exists.
   float big = -INFINITY;
-  for (int e = lane; e < E; e += 32) big = fmaxf(big, z[e]);
-  big = warp_max(big);
-  float sum = 0.f;
   for (int e = lane; e < E; e += 32) {
-    const float v = expf(z[e] - big);
-    s[e] = v;
-    sum += v;
+    const float v = z[e];
+    s[e] = v >= -FLT_MAX ? v : -FLT_MAX;
+    big = fmaxf(big, v);
   }
-  sum = warp_sum(sum);
+  big = warp_max(big);
+  float sum = 1.f;
+  if (!sigmoid) {
+    sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - big);
+    sum = warp_sum(sum);
+  }
   __syncwarp();
   float total = 0.f;
-  // A score that is no number (a row of padding may hold anything) counts as -1, below every real score and
-  // above the mark of a taken expert (-3), so that every choice names an expert that exists.
   for (int k = 0; k < top; ++k) {
-    float best = -2.f;
+    float best = -INFINITY;
     int at = E;
-    for (int e = lane; e < E; e += 32) {
-      const float v = s[e] >= 0.f || s[e] == -3.f ? s[e] : -1.f;
-      if (v > best) { best = v; at = e; }       // ascending e: the first of equals stays
-    }
+    for (int e = lane; e < E; e += 32)
+      if (s[e] > best) { best = s[e]; at = e; }       // ascending e: the first of equals stays
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
       const int oa = __shfl_xor_sync(0xffffffffu, at, o);
       if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
     }
-    const float score = best >= 0.f ? best / sum : 0.f;
+    float score = sigmoid ? 1.f / (1.f + expf(-best)) : expf(best - big) / sum;
+    if (!(score >= 0.f)) score = 0.f;
     total += score;
     if (lane == 0) {
       chosen[(size_t)t * top + k] = min(at, E - 1);
       weight[(size_t)t * top + k] = score;
-      if (at < E) s[at] = -3.f;      // taken
+      if (at < E) s[at] = -INFINITY;      // taken
     }
     __syncwarp();
   }
@@ -137,7 +143,8 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(T* __restrict__ out, co
   for (int i = threadIdx.x; i < width; i += 128) dst[i] = row ? row[i] : from_f32<T>(0.f);
 }
 
-// out[t] = sum_k weight[t, k] * y[pos_of[t, k]] (+ shared_gate[t] * shared[t]), all 32-bit.  grid (tokens).
+// out[t] = sum_k weight[t, k] * y[pos_of[t, k]] (+ shared_gate[t] * shared[t]), all 32-bit; weight null: ones.
+// grid (tokens).
 __global__ void __launch_bounds__(kThreads) moe_combine_kernel(float* __restrict__ out, const float* __restrict__ y,
                                                                const int* __restrict__ pos_of,
                                                                const float* __restrict__ weight,
@@ -152,7 +159,7 @@ __global__ void __launch_bounds__(kThreads) moe_combine_kernel(float* __restrict
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
       const int at = pos_of[(size_t)t * top + k];
-      if (at >= 0) acc = fmaf(weight[(size_t)t * top + k], y[(size_t)at * width + i], acc);
+      if (at >= 0) acc = fmaf(weight != nullptr ? weight[(size_t)t * top + k] : 1.f, y[(size_t)at * width + i], acc);
     }
     if (shared != nullptr) acc = fmaf(g, shared[(size_t)t * width + i], acc);
     out[(size_t)t * width + i] = acc;
@@ -161,11 +168,11 @@ __global__ void __launch_bounds__(kThreads) moe_combine_kernel(float* __restrict
 }  // namespace
 
 LAB_EXPORT int lab_moe_route(int* chosen, float* weight, float* shared_gate, const float* logits, int ld, int tokens,
-                             int E, int top, int gate_col, int renorm, cudaStream_t stream) {
+                             int E, int top, int gate_col, int renorm, int sigmoid, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || (size_t)kWarps * E * sizeof(float) > 48 * 1024) return (int)cudaErrorInvalidValue;
   lab_launch(moe_route_kernel, dim3((tokens + kWarps - 1) / kWarps), dim3(kThreads), sizeof(float) * kWarps * E, stream,
-             chosen, weight, shared_gate, logits, ld, tokens, E, top, gate_col, renorm);
+             chosen, weight, shared_gate, logits, ld, tokens, E, top, gate_col, renorm, sigmoid);
   LAB_LAUNCH_CHECK();
 }
 

@@ -9,7 +9,11 @@
 //                   wide, HD >= max(D, V): the entries beyond a head's own size are zeros, so that heads
 //                   whose key and value sizes differ (or are no multiple of the tensor-core tile) run on
 //                   the attention kernels built for heads of HD.  A layer that reads another layer's keys
-//                   and values has only the q part.
+//                   and values has only the q part.  Options: no norms (wq null); a rotation of the first
+//                   2 * rot_half entries of every q and k head after the norm, by position * inv_freq[i], either
+//                   of entries i and i + rot_half or of neighbours 2i and 2i + 1; and values mixed with those
+//                   an earlier layer left of the same rows, v <- (1 - mix) v + mix * v_first (v_first [tokens,
+//                   n_kv * V] floats), or left for later layers (v_keep, the same shape, before any rounding).
 //   head_gate       out[t, h, i] = attn[t, h, i] * sigmoid(g) * c, g one number per head or per entry,
 //                   read from the same projection; the V real entries of each head are packed side by
 //                   side and rounded to T for the output projection.
@@ -41,33 +45,67 @@ struct QkNormParams {
   const int* slots;
   int n_q, n_kv, D, V, HD, page_size, num_pages, has_kv, ld_q;
   float eps;
+  const int* positions;      // of the rows (rot_half > 0)
+  const float* inv_freq;
+  int rot_half, rot_pairs;
+  float* v_keep;             // or null
+  const float* v_first;      // or null
+  float v_mix;
 };
+
+// entry i of a head whose entries before the norm are `h` (weights w, or null), normed with `inv` and rotated with
+// the row's cosines and sines
+template <typename T>
+__device__ __forceinline__ float normed_rotated(const float* h, const T* w, float inv, int i, const QkNormParams& p,
+                                                const float* cs, const float* sn) {
+  const float a = w != nullptr ? h[i] * inv * to_f32(w[i]) : h[i];
+  if (i >= 2 * p.rot_half) return a;
+  const int f = p.rot_pairs ? i >> 1 : (i < p.rot_half ? i : i - p.rot_half);
+  const bool low = p.rot_pairs ? !(i & 1) : i < p.rot_half;
+  const int mate = p.rot_pairs ? i ^ 1 : (low ? i + p.rot_half : i - p.rot_half);
+  const float b = w != nullptr ? h[mate] * inv * to_f32(w[mate]) : h[mate];
+  float lo, hi;
+  rope_rotate(low ? a : b, low ? b : a, cs[f], sn[f], lo, hi);
+  return low ? lo : hi;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads) qk_norm_store_kernel(T* __restrict__ q_out, T* __restrict__ cache_k,
                                                                  T* __restrict__ cache_v, const T* __restrict__ bias,
                                                                  const T* __restrict__ wq, const T* __restrict__ wk,
                                                                  QkNormParams p) {
-  extern __shared__ float row[];      // [n_q * D + n_kv * (D + V)]
+  extern __shared__ float row[];      // [n_q * D + n_kv * (D + V)], cosines [rot_half], sines [rot_half]
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int wq_n = p.n_q * p.D, wk_n = p.has_kv ? p.n_kv * p.D : 0, wv_n = p.has_kv ? p.n_kv * p.V : 0;
   const int total = wq_n + wk_n + wv_n;
+  float *cs = row + total, *sn = cs + p.rot_half;
+  if (p.rot_half > 0) {
+    const float pos = (float)p.positions[t];
+    for (int i = threadIdx.x; i < p.rot_half; i += kThreads) sincosf(pos * p.inv_freq[i], &sn[i], &cs[i]);
+  }
   float ssq = 0.f, ssk = 0.f;
   for (int i = threadIdx.x; i < total; i += kThreads) {
     float v = sum_splits(p.proj, p.splits, p.split_stride, (size_t)t * p.ld + i);
     if (bias != nullptr) v += to_f32(bias[i]);
+    if (i < wq_n) {
+      ssq += v * v;
+    } else if (i < wq_n + wk_n) {
+      ssk += v * v;
+    } else {
+      const size_t at = (size_t)t * wv_n + i - wq_n - wk_n;
+      if (p.v_keep != nullptr) p.v_keep[at] = v;
+      if (p.v_first != nullptr) v = (1.f - p.v_mix) * v + p.v_mix * p.v_first[at];
+    }
     row[i] = v;
-    if (i < wq_n) ssq += v * v;
-    else if (i < wq_n + wk_n) ssk += v * v;
   }
   ssq = block_sum(ssq, scratch);
   const float inv_q = 1.0f / sqrtf(ssq / (float)wq_n + p.eps);
   for (int idx = threadIdx.x; idx < p.n_q * p.HD; idx += kThreads) {
     const int h = idx / p.HD, i = idx - h * p.HD;
-    const float v = i < p.D ? row[h * p.D + i] * inv_q * to_f32(wq[h * p.D + i]) : 0.f;
+    const float v = i < p.D ? normed_rotated(row + h * p.D, wq != nullptr ? wq + h * p.D : nullptr, inv_q, i, p, cs, sn) : 0.f;
     q_out[(size_t)t * p.ld_q + idx] = from_f32<T>(v);
   }
   if (!p.has_kv || cache_k == nullptr) return;
@@ -83,7 +121,8 @@ __global__ void __launch_bounds__(kThreads) qk_norm_store_kernel(T* __restrict__
   for (int idx = threadIdx.x; idx < p.n_kv * p.HD; idx += kThreads) {
     const int g = idx / p.HD, i = idx - g * p.HD;
     const size_t dst = (((size_t)page * p.n_kv + g) * p.page_size + off) * p.HD + i;
-    const float kv = i < p.D ? row[wq_n + g * p.D + i] * inv_k * to_f32(wk[g * p.D + i]) : 0.f;
+    const float kv = i < p.D ? normed_rotated(row + wq_n + g * p.D, wk != nullptr ? wk + g * p.D : nullptr, inv_k, i, p,
+                                              cs, sn) : 0.f;
     const float vv = i < p.V ? row[wq_n + wk_n + g * p.V + i] : 0.f;
     cache_k[dst] = from_f32<T>(kv);
     cache_v[dst] = from_f32<T>(vv);
@@ -113,18 +152,25 @@ int blocks_for(long long n) { return (int)((n + kThreads - 1) / kThreads < 148 *
 
 }  // namespace
 
-// proj: [splits][tokens, ld] floats (splits 1: the whole product); bias over the q, k and v columns or null.
+// proj: [splits][tokens, ld] floats (splits 1: the whole product); bias over the q, k and v columns or null; wq and wk
+// null: no norms.  rot_dims (even, at most D; 0: no rotation) entries of a head turn by positions[t] * inv_freq[i],
+// rot_pairs: neighbours, else halves.  v_keep / v_first: see above.
 LAB_EXPORT int lab_qk_norm_store(void* q_out, int ld_q, void* cache_k, void* cache_v, const float* proj, int splits,
                                  int ld, const void* bias, const void* wq, const void* wk, const int* slots, int tokens,
                                  int n_q, int n_kv, int D, int V, int HD, int page_size, int num_pages, int has_kv,
-                                 float eps, int dtype, cudaStream_t stream) {
+                                 float eps, const int* positions, const float* inv_freq, int rot_dims, int rot_pairs,
+                                 float* v_keep, const float* v_first, float v_mix, int dtype, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (HD < D || HD < V || n_q <= 0 || (has_kv && n_kv <= 0)) return (int)cudaErrorInvalidValue;
+  if (rot_dims < 0 || rot_dims % 2 || rot_dims > D || (rot_dims > 0 && (positions == nullptr || inv_freq == nullptr)) ||
+      (!has_kv && (v_keep != nullptr || v_first != nullptr)) || (has_kv && (wq == nullptr) != (wk == nullptr)))
+    return (int)cudaErrorInvalidValue;
   QkNormParams p;
   p.proj = proj; p.splits = splits; p.split_stride = (long long)tokens * ld; p.ld = ld; p.slots = slots;
   p.n_q = n_q; p.n_kv = n_kv; p.D = D; p.V = V; p.HD = HD; p.page_size = page_size; p.num_pages = num_pages;
-  p.has_kv = has_kv; p.ld_q = ld_q; p.eps = eps;
-  const size_t smem = (size_t)(n_q * D + (has_kv ? n_kv * (D + V) : 0)) * sizeof(float);
+  p.has_kv = has_kv; p.ld_q = ld_q; p.eps = eps; p.positions = positions; p.inv_freq = inv_freq;
+  p.rot_half = rot_dims / 2; p.rot_pairs = rot_pairs; p.v_keep = v_keep; p.v_first = v_first; p.v_mix = v_mix;
+  const size_t smem = (size_t)(n_q * D + (has_kv ? n_kv * (D + V) : 0) + rot_dims) * sizeof(float);
   if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   if (dtype == LAB_F32) {
     if (smem > 48 * 1024)

@@ -203,6 +203,15 @@ __device__ __forceinline__ float silu_gate(float g, float u, float limit) {
   }
   return silu_gate(g, u);
 }
+// The same by the gate's activation: 1, the tanh form of GELU of g, times u, with 0.5 (1 + tanh(y)) written as the
+// sigmoid of 2 y; 0, as above.
+__device__ __forceinline__ float gate_value(float g, float u, int act, float limit) {
+  if (act == 1) {
+    const float twice = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+    return __fdividef(g, 1.f + __expf(-twice)) * u;
+  }
+  return silu_gate(g, u, limit);
+}
 
 // ---- host: tensor maps -----------------------------------------------------------------------
 typedef CUresult (*LabEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,

@@ -267,9 +267,9 @@ def rope_kv_write_table(qkv, table, rotary_dim, slots, cache_k, cache_v, n_q, n_
 
 def gemm_plain(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, gated: bool = False,
                out_f32: bool = False, out: torch.Tensor | None = None, gelu: bool = False,
-               gate_limit: float = 0.0) -> torch.Tensor:
+               gate_limit: float = 0.0, gate_act: str = "silu") -> torch.Tensor:
     """out = x @ w.T (+ bias) on the ordinary arithmetic units; `gated`: silu(x@wg.T) * (x@wu.T), w = [wg; wu]
-    (`gate_limit` > 0: the capped form, see `linear_gated`); `gelu`: the tanh form of GELU after the bias, before
+    (`gate_limit`, `gate_act`: see `linear_gated`); `gelu`: the tanh form of GELU after the bias, before
     the rounding."""
     assert not (gated and gelu)
     _on_gpu(x, w, bias, out)
@@ -282,7 +282,8 @@ def gemm_plain(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = Non
         out = torch.empty((M, N), dtype=odt, device=x.device)
     assert out.dtype == odt and out.stride(1) == 1 and out.shape == (M, N)
     _check(lib("gemm_plain").lab_gemm_plain(_ptr(out), _ptr(x), _ptr(w), _ptr(bias), M, N, K, x.stride(0),
-                                            out.stride(0), (1 + int(gelu)) if gelu else int(gated), dtype_code(x.dtype), int(out_f32),
+                                            out.stride(0), _epilogue(gated, gelu, gate_act, gate_limit), dtype_code(x.dtype),
+                                            int(out_f32),
                                             ctypes.c_float(gate_limit), _stream()),
            "gemm_plain")
     return out
@@ -414,7 +415,8 @@ def force_plain(flag: bool) -> bool:
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, gated: bool = False,
             out_f32: bool = False, swap: bool | None = None, bn: int | None = None, splits: int = 1,
-            out: torch.Tensor | None = None, gelu: bool = False, gate_limit: float = 0.0) -> torch.Tensor:
+            out: torch.Tensor | None = None, gelu: bool = False, gate_limit: float = 0.0,
+            gate_act: str = "silu") -> torch.Tensor:
     """out = x @ w.T (+ bias) on the tcgen05 tensor cores (bfloat16 in, 32-bit accumulate); `gelu`: the
     tanh form of GELU after the bias, before the rounding (not with `gated` or `splits`).
 
@@ -457,14 +459,14 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, 
     if gelu and (gated or splits > 1):
         raise KernelError("gemm_tc: GELU goes with the plain, unsplit product")
     _check(lib("gemm_tc").lab_gemm_tc(_ptr(out), _ptr(x), _ptr(w), _ptr(bias), T, n_out, K, x.stride(0), ld_out,
-                                      (1 + int(gelu)) if gelu else int(gated), int(f32), int(swap), bn, splits,
+                                      _epilogue(gated, gelu, gate_act, gate_limit), int(f32), int(swap), bn, splits,
                                       ctypes.c_float(gate_limit), _stream()), "gemm_tc")
     return out
 
 
 def gemm_tc2(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, gated: bool = False,
              out_f32: bool = False, splits: int = 1, out: torch.Tensor | None = None, bn: int = 0,
-             gelu: bool = False, gate_limit: float = 0.0) -> torch.Tensor:
+             gelu: bool = False, gate_limit: float = 0.0, gate_act: str = "silu") -> torch.Tensor:
     """out = x @ w.T (+ bias) on pairs of SMs (tcgen05.mma.cta_group::2): tiles of 256 tokens by 256
     accumulator columns, each CTA of a pair loading half of the weight tile.  For steps with many
     tokens; `splits` > 1 returns 32-bit partial products [splits, tokens, out].  `bn`: accumulator
@@ -494,7 +496,7 @@ def gemm_tc2(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
     if gelu and (gated or splits > 1):
         raise KernelError("gemm_tc2: GELU goes with the plain, unsplit product")
     _check(lib("gemm_tc2").lab_gemm_tc2(_ptr(out), _ptr(x), _ptr(w), _ptr(bias), T, n_out, K, x.stride(0), ld_out,
-                                        (1 + int(gelu)) if gelu else int(gated), int(f32), splits, bn,
+                                        _epilogue(gated, gelu, gate_act, gate_limit), int(f32), splits, bn,
                                         ctypes.c_float(gate_limit), _stream()), "gemm_tc2")
     return out
 
@@ -630,6 +632,18 @@ def _tc_operands(x, w) -> bool:
 
 # activations a plain product applies in its epilogue, with their codes (`gelu` = 1, 2 in the product kernels' faces)
 ACTIVATIONS = {"gelu_tanh": 1, "relu2": 2}
+# activations of a gated pair of products, with the code the product kernels' faces take as `gated`
+GATE_ACTIVATIONS = {"silu": 1, "gelu_tanh": 4}
+
+
+def _epilogue(gated: bool, gelu: int, gate_act: str, gate_limit: float) -> int:
+    """The epilogue's code in the product kernels' faces: 0 none, 2 and 3 an activation of the plain product, 1 and
+    4 a gated pair."""
+    if not gated:
+        return 1 + int(gelu) if gelu else 0
+    if gate_act not in GATE_ACTIVATIONS or (gate_limit > 0.0 and gate_act != "silu"):
+        raise KernelError(f"gated product: activation {gate_act!r} is not built (or not with a limit)")
+    return GATE_ACTIVATIONS[gate_act]
 
 
 def linear(x, w, bias=None, out_f32=False, allow_partial=False, out=None, act=None):
@@ -658,18 +672,19 @@ def linear(x, w, bias=None, out_f32=False, allow_partial=False, out=None, act=No
     return gemm_tc(x, w, bias, out_f32=out_f32, out=out, gelu=gelu)
 
 
-def linear_gated(x, w_gate_up, limit: float = 0.0):
-    """silu(g) * u with g = x @ wg.T, u = x @ wu.T and w_gate_up = [wg; wu].  `limit` > 0: the capped form,
-    g' = min(g, limit), u' = clamp(u, -limit, limit), g' * sigmoid(1.702 g') * (u' + 1)."""
+def linear_gated(x, w_gate_up, limit: float = 0.0, act: str = "silu"):
+    """act(g) * u with g = x @ wg.T, u = x @ wu.T and w_gate_up = [wg; wu]; `act` "silu" or "gelu_tanh" (the tanh
+    form of GELU).  `limit` > 0 (with "silu"): the capped form, g' = min(g, limit), u' = clamp(u, -limit, limit),
+    g' * sigmoid(1.702 g') * (u' + 1)."""
     if x.dtype == torch.float32 or _force_plain or not _tc_operands(x, w_gate_up):
-        return gemm_plain(x, w_gate_up, None, gated=True, gate_limit=limit)
+        return gemm_plain(x, w_gate_up, None, gated=True, gate_limit=limit, gate_act=act)
     # Pairs of SMs (256 tokens x 128 features per tile, gate rows in one CTA and up rows in the other)
     # once their tiles fill most of the 74 pairs: measured 6 to 12 % faster from there on at the 0.5B,
     # 1.5B and 7B layer sizes (2,048 tokens: 31.7 against 33.7, 76 against 85, 349 against 385 us).
     T, inter = x.shape[0], w_gate_up.shape[0] // 2
     if -(-T // 256) * (-(-inter // 128)) >= 64:
-        return gemm_tc2(x, w_gate_up, None, gated=True, gate_limit=limit)
-    return gemm_tc(x, w_gate_up, None, gated=True, gate_limit=limit)
+        return gemm_tc2(x, w_gate_up, None, gated=True, gate_limit=limit, gate_act=act)
+    return gemm_tc(x, w_gate_up, None, gated=True, gate_limit=limit, gate_act=act)
 
 
 # Which kernel serves requests that bring several tokens: "auto" (tcgen05 for heads of 64 and of 128
@@ -1222,21 +1237,34 @@ def padded_head(dim: int, vdim: int) -> int:
     return (max(dim, vdim) + 15) // 16 * 16
 
 
-def qk_norm_store(proj: torch.Tensor, bias, w_q: torch.Tensor, w_k, slots, cache_k, cache_v, n_q: int, n_kv: int,
-                  dim: int, vdim: int, head: int, eps: float, has_kv: bool = True) -> torch.Tensor:
+def qk_norm_store(proj: torch.Tensor, bias, w_q, w_k, slots, cache_k, cache_v, n_q: int, n_kv: int,
+                  dim: int, vdim: int, head: int, eps: float, has_kv: bool = True, dtype: torch.dtype | None = None,
+                  positions: torch.Tensor | None = None, inv_freq: torch.Tensor | None = None, rot_dims: int = 0,
+                  rot_pairs: bool = False, v_keep: torch.Tensor | None = None, v_first: torch.Tensor | None = None,
+                  v_mix: float = 0.0) -> torch.Tensor:
     """From the 32-bit fused projection `proj` [tokens, >= q + k + v columns] (or split-K partial products
     [splits, tokens, ...]) and an optional bias over those columns: q and k RMS-normed over their whole
     projections with the weights `w_q`, `w_k`; q returned [tokens, n_q * head] in the weights' storage type,
     heads padded with zeros to `head` entries; k and v written the same way into their cache slots
-    (`cache_k` None: nothing is written).  `has_kv` False: the projection holds q only."""
-    _on_gpu(proj, bias, w_q, w_k, slots, cache_k, cache_v)
+    (`cache_k` None: nothing is written).  `has_kv` False: the projection holds q only.  `w_q` and `w_k` None: no
+    norms, `dtype` then names the storage type.  `rot_dims` > 0: after the norm the first that many entries of every q
+    and k head turn by position * inv_freq[i], entries i and i + rot_dims / 2 together (`rot_pairs`: 2i and 2i + 1).
+    `v_keep` [tokens, n_kv * vdim] 32-bit receives the values as projected; `v_first` of the same shape is mixed into
+    them, v <- (1 - v_mix) v + v_mix v_first, before they are stored."""
+    _on_gpu(proj, bias, w_q, w_k, slots, cache_k, cache_v, positions, inv_freq, v_keep, v_first)
     splits = proj.shape[0] if proj.dim() == 3 else 1
     tokens, ld = proj.shape[-2], proj.stride(-2)       # a column slice of a wider product will do
     assert proj.dtype == torch.float32 and proj.stride(-1) == 1 and (splits == 1 or proj.stride(0) == tokens * ld)
     need = n_q * dim + (n_kv * (dim + vdim) if has_kv else 0)
-    assert proj.shape[-1] >= need and w_q.numel() == n_q * dim and (not has_kv or w_k.numel() == n_kv * dim)
-    assert bias is None or (bias.numel() >= need and bias.dtype == w_q.dtype)
-    dt = w_q.dtype
+    assert proj.shape[-1] >= need and (w_q is None or w_q.numel() == n_q * dim)
+    assert not has_kv or (w_k is None if w_q is None else w_k.numel() == n_kv * dim)
+    dt = w_q.dtype if w_q is not None else dtype
+    assert dt is not None and (dtype is None or dtype == dt)
+    assert bias is None or (bias.numel() >= need and bias.dtype == dt)
+    assert rot_dims == 0 or (positions.dtype == torch.int32 and positions.numel() >= tokens and
+                             inv_freq.dtype == torch.float32 and inv_freq.numel() >= rot_dims // 2)
+    for t in (v_keep, v_first):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape) == (tokens, n_kv * vdim))
     page_size = num_pages = 0
     if cache_k is not None:
         num_pages, kvh, page_size, d = cache_k.shape
@@ -1246,7 +1274,8 @@ def qk_norm_store(proj: torch.Tensor, bias, w_q: torch.Tensor, w_k, slots, cache
     _check(lib("norm_attention").lab_qk_norm_store(
         _ptr(q), q.stride(0), _ptr(cache_k), _ptr(cache_v), _ptr(proj), splits, ld, _ptr(bias), _ptr(w_q), _ptr(w_k),
         _ptr(slots), tokens, n_q, n_kv, dim, vdim, head, page_size, num_pages, int(has_kv), ctypes.c_float(eps),
-        dtype_code(dt), _stream()), "qk_norm_store")
+        _ptr(positions), _ptr(inv_freq), int(rot_dims), int(bool(rot_pairs)), _ptr(v_keep), _ptr(v_first),
+        ctypes.c_float(v_mix), dtype_code(dt), _stream()), "qk_norm_store")
     return q
 
 
@@ -1463,10 +1492,15 @@ def selective_scan(x: torch.Tensor, dt_pre: torch.Tensor, bc: torch.Tensor, b_at
 # ----------------------------------------------------------------------------------------
 # Routed feed-forward layers (csrc/kernels/moe.cu and the grouped products).
 # ----------------------------------------------------------------------------------------
-def moe_route(logits: torch.Tensor, experts: int, top: int, gate_col: int = -1, renorm: bool = True):
+MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
+def moe_route(logits: torch.Tensor, experts: int, top: int, gate_col: int = -1, renorm: bool = True,
+              score: str = "softmax"):
     """From 32-bit router logits [tokens, >= experts] (column `gate_col` >= 0: the logit of a shared expert's
     gate): (chosen experts [tokens, top] int32, their weights [tokens, top], sigmoid of the gate's logit
-    [tokens] or None).  The weights are the chosen scores over their sum, or (`renorm` False) as they are."""
+    [tokens] or None).  The scores are the softmax over all experts or (`score` "sigmoid") the sigmoid of each
+    logit; the weights are the chosen scores over their sum, or (`renorm` False) as they are."""
     _on_gpu(logits)
     tokens = logits.shape[0]
     assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= experts
@@ -1474,7 +1508,8 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, gate_col: int = -1, 
     weight = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     gate = torch.empty((tokens,), dtype=torch.float32, device=logits.device) if gate_col >= 0 else None
     _check(lib("moe").lab_moe_route(_ptr(chosen), _ptr(weight), _ptr(gate), _ptr(logits), logits.stride(0), tokens,
-                                    experts, top, gate_col, int(bool(renorm)), _stream()), "moe_route")
+                                    experts, top, gate_col, int(bool(renorm)), MOE_SCORES[score], _stream()),
+           "moe_route")
     return chosen, weight, gate
 
 
@@ -1497,13 +1532,14 @@ def moe_align(chosen: torch.Tensor, experts: int, tile: int):
     return row_src, tile_group, pos_of
 
 
-def moe_combine(y: torch.Tensor, pos_of: torch.Tensor, weight: torch.Tensor, shared: torch.Tensor | None,
-                shared_gate: torch.Tensor | None) -> torch.Tensor:
-    """out[t] = sum_k weight[t, k] * y[pos_of[t, k]] (+ shared_gate[t] * shared[t]), 32-bit."""
+def moe_combine(y: torch.Tensor, pos_of: torch.Tensor, weight: torch.Tensor | None, shared: torch.Tensor | None,
+                shared_gate: torch.Tensor | None, top: int | None = None) -> torch.Tensor:
+    """out[t] = sum_k weight[t, k] * y[pos_of[t, k]] (+ shared_gate[t] * shared[t]), 32-bit.  `weight` None: the plain
+    sum over each token's `top` pairs."""
     _on_gpu(y, pos_of, weight, shared, shared_gate)
-    tokens, top = weight.shape
+    tokens, top = weight.shape if weight is not None else (pos_of.numel() // top, top)
     width = y.shape[1]
-    assert y.dtype == torch.float32 and y.is_contiguous() and weight.dtype == torch.float32
+    assert y.dtype == torch.float32 and y.is_contiguous() and (weight is None or weight.dtype == torch.float32)
     assert shared is None or (shared.dtype == torch.float32 and shared.is_contiguous() and shared.shape == (tokens, width))
     out = torch.empty((tokens, width), dtype=torch.float32, device=y.device)
     _check(lib("moe").lab_moe_combine(_ptr(out), _ptr(y), _ptr(pos_of), _ptr(weight), _ptr(shared), _ptr(shared_gate),
@@ -1556,12 +1592,15 @@ def moe_gather(x: torch.Tensor, row_src: torch.Tensor, top: int) -> torch.Tensor
 
 
 def linear_grouped_tc(x: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, gated: bool = False,
-                      out_f32: bool = False, bn: int | None = None, gate_limit: float = 0.0) -> torch.Tensor:
+                      out_f32: bool = False, bn: int | None = None, gate_limit: float = 0.0, gate_act: str = "silu",
+                      row_scale: torch.Tensor | None = None, row_src: torch.Tensor | None = None) -> torch.Tensor:
     """Row r of the result is x[r] times the matrix w[tile_group[r // 128]] transposed, on the tcgen05 tensor cores;
     x [rows, K] bfloat16 with rows a multiple of 128, w as for `linear_grouped`.  Rows of tiles whose group is -1
-    are left unwritten."""
-    _on_gpu(x, w, tile_group)
+    are left unwritten.  `row_scale` (with `gated`; 32-bit, by pair): row r counts as row_scale[row_src[r]] * x[r]."""
+    _on_gpu(x, w, tile_group, row_scale, row_src)
     rows, K = x.shape
+    assert row_scale is None or (gated and row_scale.dtype == torch.float32 and row_scale.is_contiguous() and
+                                 row_src.numel() == rows)
     N = w.shape[1] // 2 if gated else w.shape[1]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not _tc_operands(x, w[0]) or w.shape[2] != K:
         raise KernelError("linear_grouped_tc takes bfloat16 operands with rows of whole 16-byte units")
@@ -1570,21 +1609,24 @@ def linear_grouped_tc(x: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor
     if bn is None:
         bn = 256 if gated else 128
     _check(lib("gemm_tc").lab_gemm_tc_grouped(_ptr(out), _ptr(x), _ptr(w), rows, N, K, x.stride(0), out.stride(0),
-                                              int(gated), int(out_f32), bn, w.shape[0], _ptr(tile_group),
-                                              ctypes.c_float(gate_limit), _stream()),
+                                              _epilogue(gated, 0, gate_act, gate_limit), int(out_f32), bn, w.shape[0],
+                                              _ptr(tile_group), ctypes.c_float(gate_limit), _ptr(row_scale),
+                                              _ptr(row_src if row_scale is not None else None), _stream()),
            "gemm_tc_grouped")
     return out
 
 
-def moe_experts_up(x: torch.Tensor, w_gate_up: torch.Tensor, lay: MoeLayout, top: int, limit: float = 0.0) -> torch.Tensor:
-    """silu(W_gate h) * (W_up h) of every pair's token with its expert's matrices, [rows, expert_ff] in the layout
-    (`limit` > 0: the capped form of the gate, see `linear_gated`)."""
+def moe_experts_up(x: torch.Tensor, w_gate_up: torch.Tensor, lay: MoeLayout, top: int, limit: float = 0.0,
+                   act: str = "silu", in_scale: torch.Tensor | None = None) -> torch.Tensor:
+    """act(W_gate h) * (W_up h) of every pair's token with its expert's matrices, [rows, expert_ff] in the layout
+    (`limit`, `act`: see `linear_gated`).  `in_scale` [tokens, top] 32-bit: a pair's expert reads in_scale * h (both
+    products are scaled where they leave in 32-bit, so the scaled h is never rounded)."""
+    more = {"gated": True, "gate_limit": limit, "gate_act": act, "row_scale": in_scale}
     if lay.tc:
-        return linear_grouped_tc(moe_gather(x, lay.row_src, top), w_gate_up, lay.tile_group, gated=True, gate_limit=limit)
+        return linear_grouped_tc(moe_gather(x, lay.row_src, top), w_gate_up, lay.tile_group, row_src=lay.row_src, **more)
     if lay.few:
-        return linear_grouped_few(x, w_gate_up, lay.row_src, top, True, lay.tile_group, lay.tile, gated=True,
-                                  gate_limit=limit)
-    return linear_grouped(x, w_gate_up, lay.row_src, top, lay.tile_group, lay.rows, gated=True, gate_limit=limit)
+        return linear_grouped_few(x, w_gate_up, lay.row_src, top, True, lay.tile_group, lay.tile, **more)
+    return linear_grouped(x, w_gate_up, lay.row_src, top, lay.tile_group, lay.rows, **more)
 
 
 def moe_experts_down(act: torch.Tensor, w_down: torch.Tensor, lay: MoeLayout) -> torch.Tensor:
@@ -1598,10 +1640,12 @@ def moe_experts_down(act: torch.Tensor, w_down: torch.Tensor, lay: MoeLayout) ->
 
 def linear_grouped_few(x: torch.Tensor, w: torch.Tensor, row_src: torch.Tensor, row_div: int, gather: bool,
                        tile_group: torch.Tensor, tile: int, gated: bool = False, out_f32: bool = False,
-                       gate_limit: float = 0.0) -> torch.Tensor:
+                       gate_limit: float = 0.0, gate_act: str = "silu",
+                       row_scale: torch.Tensor | None = None) -> torch.Tensor:
     """`linear_grouped` for a handful of rows: only rows whose `row_src` is not -1 are formed (the others stay
     unwritten); `gather`: row r reads x[row_src[r] // row_div], else x[r]."""
-    _on_gpu(x, w, row_src, tile_group)
+    _on_gpu(x, w, row_src, tile_group, row_scale)
+    assert row_scale is None or (gated and row_scale.dtype == torch.float32 and row_scale.is_contiguous())
     rows, K = row_src.numel(), x.shape[1]
     N = w.shape[1] // 2 if gated else w.shape[1]
     assert w.is_contiguous() and w.dim() == 3 and w.shape[2] == K and w.dtype == x.dtype and x.stride(1) == 1
@@ -1609,9 +1653,10 @@ def linear_grouped_few(x: torch.Tensor, w: torch.Tensor, row_src: torch.Tensor, 
     odt = torch.float32 if (out_f32 or x.dtype == torch.float32) else x.dtype
     out = torch.empty((rows, N), dtype=odt, device=x.device)
     _check(lib("gemm_plain").lab_gemm_plain_grouped_few(
-        _ptr(out), _ptr(x), _ptr(w), rows, N, K, x.stride(0), out.stride(0), int(gated),
+        _ptr(out), _ptr(x), _ptr(w), rows, N, K, x.stride(0), out.stride(0), _epilogue(gated, 0, gate_act, gate_limit),
         ctypes.c_longlong(w.shape[1] * K), _ptr(row_src), int(row_div), int(gather), _ptr(tile_group), int(tile),
-        dtype_code(x.dtype), int(out_f32), ctypes.c_float(gate_limit), _stream()), "gemm_plain_grouped_few")
+        dtype_code(x.dtype), int(out_f32), ctypes.c_float(gate_limit), _ptr(row_scale), _stream()),
+        "gemm_plain_grouped_few")
     return out
 
 
@@ -1622,11 +1667,16 @@ def grouped_tile_rows() -> int:
 
 def linear_grouped(x: torch.Tensor, w: torch.Tensor, row_src: torch.Tensor | None, row_div: int,
                    tile_group: torch.Tensor, rows: int, gated: bool = False, out_f32: bool = False,
-                   gate_limit: float = 0.0) -> torch.Tensor:
+                   gate_limit: float = 0.0, gate_act: str = "silu",
+                   row_scale: torch.Tensor | None = None) -> torch.Tensor:
     """Row r of the result is x[row_src[r] // row_div] (row_src None: x[r]) times the matrix w[tile_group[r // tile]]
     transposed; w [groups, out, in], with `gated` [groups, 2 * out, in] (gate rows, then up rows) and the result
-    silu(gate) * up.  Rows of tiles whose group is -1 are left unwritten; rows whose source is -1 read zeros."""
-    _on_gpu(x, w, row_src, tile_group)
+    silu(gate) * up (`gate_act`, `gate_limit`: see `linear_gated`).  Rows of tiles whose group is -1 are left
+    unwritten; rows whose source is -1 read zeros.  `row_scale` (with `gated`; 32-bit, by pair): row r counts as
+    row_scale[row_src[r]] times the row it reads."""
+    _on_gpu(x, w, row_src, tile_group, row_scale)
+    assert row_scale is None or (gated and row_src is not None and row_scale.dtype == torch.float32 and
+                                 row_scale.is_contiguous())
     K = x.shape[1]
     N = w.shape[1] // 2 if gated else w.shape[1]
     assert w.is_contiguous() and w.dim() == 3 and w.shape[2] == K and w.dtype == x.dtype and x.stride(1) == 1
@@ -1634,9 +1684,9 @@ def linear_grouped(x: torch.Tensor, w: torch.Tensor, row_src: torch.Tensor | Non
     odt = torch.float32 if (out_f32 or x.dtype == torch.float32) else x.dtype
     out = torch.empty((rows, N), dtype=odt, device=x.device)
     _check(lib("gemm_plain").lab_gemm_plain_grouped(
-        _ptr(out), _ptr(x), _ptr(w), rows, N, K, x.stride(0), out.stride(0), int(gated),
+        _ptr(out), _ptr(x), _ptr(w), rows, N, K, x.stride(0), out.stride(0), _epilogue(gated, 0, gate_act, gate_limit),
         ctypes.c_longlong(w.shape[1] * K), _ptr(row_src), int(row_div), _ptr(tile_group), dtype_code(x.dtype),
-        int(out_f32), ctypes.c_float(gate_limit), _stream()), "gemm_plain_grouped")
+        int(out_f32), ctypes.c_float(gate_limit), _ptr(row_scale), _stream()), "gemm_plain_grouped")
     return out
 
 

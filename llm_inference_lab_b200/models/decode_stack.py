@@ -37,7 +37,8 @@ def _fits(block, dtype) -> bool:
     if type(block) is not PreNormBlock or dtype != torch.bfloat16:
         return False
     m, f = block.mixer, block.ffn
-    if type(m) is not GQAttention or type(f) is not GatedMLP or any(type(n) is not RMSNorm for n in block.norms):
+    if (type(m) is not GQAttention or type(f) is not GatedMLP or f.act != "silu"
+            or any(type(n) is not RMSNorm for n in block.norms)):
         return False
     if type(m.position) is not Rope or m.position.rotary_dim != m.d or m.d not in (64, 128) or m.b_o is not None:
         return False

@@ -124,7 +124,7 @@ class HyperStreamBlock(Block):
         if x.dim() == 2:       # the embedding output: every stream starts as a copy of it
             if pending is not None:
                 raise ValueError("hyper_stream: a sum is owed to rows that are not streams yet")
-            x = ops.hyper_expand(x, self.streams)
+            x = ops.hyper_expand(x, self.streams) if self.streams > 1 else x.view(x.shape[0], 1, x.shape[1])
         elif x.shape[1] != self.streams:
             raise ValueError("hyper_stream: the number of streams changed between layers")
         (in1, out1, mix1), n1 = self.coef[0], self.norms[0]

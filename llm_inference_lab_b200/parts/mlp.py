@@ -10,11 +10,11 @@ from .spec import PartSpec, TensorSpec
 
 class GatedMLP(FeedForward):
     """down( act(x Wg^T) * (x Wu^T) ), no biases; act is SiLU
-    (rust/engine/src/runner/model/qwen2/kernels.rs:1469-1486, engine.rs:1242-1293).
+    (rust/engine/src/runner/model/qwen2/kernels.rs:1469-1486, engine.rs:1242-1293) or "gelu_tanh", the tanh form of GELU.
     Gate and up matrices are concatenated at load time; the activation and the product are
     the epilogue of their matrix product."""
 
-    ACTS = ("silu",)
+    ACTS = ("silu", "gelu_tanh")
     NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
 
     @classmethod
@@ -38,9 +38,10 @@ class GatedMLP(FeedForward):
         # True: the product leaves in 32-bit (whole, or as split-K partial sums), for a block whose
         # residual stream is 32-bit
         self.out_f32 = bool(spec.get("out_f32"))
+        self.act = spec["act"]
 
     def forward(self, x, ctx):
-        act = ops.linear_gated(x, self.w_gate_up)
+        act = ops.linear_gated(x, self.w_gate_up, act=self.act)
         return ops.linear(act, self.w_down, None, out_f32=self.out_f32, allow_partial=True)
 
 

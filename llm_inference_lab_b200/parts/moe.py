@@ -12,7 +12,8 @@ class RoutedExperts(FeedForward):
     """`experts` gated feed-forwards W_down (silu(W_gate h) * (W_up h)) of `expert_ff` rows, without biases, of
     which every token uses `top`: router logits z = W_router h in 32-bit, scores softmax(z) over all experts,
     the `top` largest chosen (ties: the smaller index), weighted by their scores over the sum of the chosen
-    scores (+ 1e-20).  `shared_ff` > 0: one more expert of that many rows runs for every token and is added,
+    scores (+ 1e-20).  `score` "sigmoid": scores sigmoid(z), one expert's apart from the others'.  `scale_input` True:
+    a weight multiplies its expert's input instead of its output, the result is the sum of expert(w * h).  `shared_ff` > 0: one more expert of that many rows runs for every token and is added,
     with `shared_gate` multiplied by sigmoid(W_sg h), one number per token.  `renorm` False: the weights are the
     chosen scores as they are.  `limit` > 0 (and `shared_limit` for the shared expert): the experts are of the
     capped form W_down (g' * sigmoid(1.702 g') * (u' + 1)) with g' = min(W_gate h, limit) and u' = clamp(W_up h,
@@ -60,6 +61,10 @@ class RoutedExperts(FeedForward):
         self.shared_ff = int(spec.get("shared_ff") or 0)
         self.gated_share = bool(self.shared_ff and spec.get("shared_gate"))
         self.renorm = bool(spec.get("renorm", True))
+        self.score = spec.get("score", "softmax")
+        if self.score not in ops.MOE_SCORES:
+            raise ValueError(f"routed_experts: score {self.score!r} is not one of {tuple(ops.MOE_SCORES)}")
+        self.scale_input = bool(spec.get("scale_input"))
         self.limit, self.shared_limit = float(spec.get("limit") or 0.0), float(spec.get("shared_limit") or 0.0)
         rows = [w(n["router"])] + ([w(n["shared_gate"]).reshape(1, -1)] if self.gated_share else [])
         self.w_router = torch.cat(rows, dim=0).contiguous()
@@ -74,15 +79,17 @@ class RoutedExperts(FeedForward):
     def forward(self, x, ctx):
         E, top = self.experts, self.top
         logits = ops.linear(x, self.w_router, None, out_f32=True)
-        chosen, weight, gate = ops.moe_route(logits, E, top, gate_col=E if self.gated_share else -1, renorm=self.renorm)
+        chosen, weight, gate = ops.moe_route(logits, E, top, gate_col=E if self.gated_share else -1, renorm=self.renorm,
+                                             score=self.score)
         lay = ops.moe_layout(chosen, E, x.dtype, x.shape[1], self.ff)
-        act = ops.moe_experts_up(x, self.w_gate_up, lay, top, limit=self.limit)
+        act = ops.moe_experts_up(x, self.w_gate_up, lay, top, limit=self.limit,
+                                 in_scale=weight if self.scale_input else None)
         y = ops.moe_experts_down(act, self.w_down, lay)
         shared = None
         if self.shared_ff:
             shared = ops.linear(ops.linear_gated(x, self.w_shared_gate_up, limit=self.shared_limit), self.w_shared_down,
                                 None, out_f32=True)
-        return ops.moe_combine(y, lay.pos_of, weight, shared, gate)
+        return ops.moe_combine(y, lay.pos_of, None if self.scale_input else weight, shared, gate, top=top)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

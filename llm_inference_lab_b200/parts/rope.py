@@ -1,11 +1,30 @@
 """Rotary position encoding (split-half pairing) with a theta parameter."""
 from __future__ import annotations
 
+import math
+
 import numpy as np
 import torch
 
 from ..kernels import ops
 from .base import PositionEncoding, register_part
+
+
+def rope_frequencies(base: float, dims: int, divide: float = 1.0, bands=None) -> np.ndarray:
+    """base^(-2i / dims) for i < dims / 2, formed in 64-bit and rounded once to 32-bit.  `divide`: every frequency is
+    divided by it.  `bands` (factor, low, high, original), for contexts stretched beyond `original` positions: a
+    frequency f whose wavelength 2 pi / f is longer than original / low is divided by factor, one shorter than
+    original / high stays as it is, and between the two, with s = (original / wavelength - low) / (high - low), it
+    becomes (1 - s) f / factor + s f."""
+    i = np.arange(dims // 2, dtype=np.float64)
+    f = np.power(float(base), -2.0 * i / max(dims, 1)) / float(divide)
+    if bands is not None:
+        factor, low, high, original = (float(b) for b in bands)
+        wave = 2.0 * math.pi / f
+        blend = (original / wave - low) / (high - low) if high != low else np.zeros_like(f)
+        f = np.where(wave < original / high, f,
+                     np.where(wave > original / low, f / factor, (1.0 - blend) * f / factor + blend * f))
+    return f.astype(np.float32)
 
 
 class Rope(PositionEncoding):
@@ -18,10 +37,8 @@ class Rope(PositionEncoding):
     def __init__(self, spec, weights, dtype, device):
         super().__init__(spec, weights, dtype, device)
         self.rotary_dim = int(spec["rotary_dim"])
-        i = np.arange(self.rotary_dim // 2, dtype=np.float64)
-        inv = np.power(float(spec["theta"]), -2.0 * i / self.rotary_dim).astype(np.float32)
         self.theta = float(spec["theta"])
-        self.inv_freq = torch.from_numpy(inv).to(device)
+        self.inv_freq = torch.from_numpy(rope_frequencies(self.theta, self.rotary_dim)).to(device)
 
     def table(self, positions, scratch):
         """(cos, sin) of every row's angles [tokens, rotary_dim / 2, 2] in 32-bit, formed once per step

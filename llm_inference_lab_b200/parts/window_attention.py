@@ -1,15 +1,15 @@
-"""Grouped-query attention with rotary positions on neighbouring pairs, a window that keeps the first tokens,
-a softmax with one more (or a learned term) in its denominator, and, as options, a norm per head on q and k,
-temperatures on q, and a learned bias by distance."""
+"""Grouped-query attention with rotary positions, a window that may keep the first tokens, a softmax with one more
+(or a learned term) in its denominator, and, as options, norms on q and k (per head or over the whole projections),
+temperatures on q, a learned bias by distance, and values mixed with an earlier layer's."""
 from __future__ import annotations
 
 import math
 
-import numpy as np
 import torch
 
 from ..kernels import ops
 from .base import CacheView, Mixer, StepContext, register_part
+from .rope import rope_frequencies
 from .spec import PagedKV, PartSpec, TensorSpec
 
 
@@ -45,7 +45,14 @@ class PairRopeAttention(Mixer):
     a value.  W_o closes.
 
     Further options, each off unless named:
+    `rot_layout` "halves": entries i and i + rot_dims / 2 of a head turn together instead of neighbours.
     `rot_scaling`: every rotation frequency is divided by this factor (positions stretched linearly).
+    `rot_bands` (factor, low, high, original): frequencies scaled by their wavelength (see `rope_frequencies`).
+    `proj_norm`: before the rotation q and k are RMS-normed over their whole projections, all heads at once, with
+    plain weights (tensors `q.norm` [heads * dim], `k.norm` [kv_heads * dim]; `eps` inside the root).
+    `v_mix`: "first", the layer leaves its values for later layers of the same step; "mix", v <- (1 - lambda) v +
+    lambda v_first with a learned number lambda (tensor `vmix`, which the "first" layer stores without using it) and
+    the values v_first the "first" layer left for the same token, before they are cached.
     `head_norm` "unit": after the rotation every q and k head is divided by its root mean square over `dim`
     (`eps` inside the root); "weight": and multiplied by a weight of `dim` entries shared by all heads (tensors
     `q.norm`, `k.norm`).
@@ -59,7 +66,8 @@ class PairRopeAttention(Mixer):
     the last row at `far`.
 
     One product forms q, k (and v) in 32-bit; one kernel adds the biases, rotates, norms, applies the
-    temperatures, rounds q and writes k and v to their page slots.  Heads are cached `ops.padded_head(dim, vdim)`
+    temperatures, mixes values, rounds q and writes k and v to their page slots (a block per row where whole
+    projections are normed, halves turn or values mix; there is no norm per head and no temperature then).  Heads are cached `ops.padded_head(dim, vdim)`
     wide with zeros beyond their own size.  `forward_inner` leaves the heads' outputs for a caller that owns the
     output projection (mixers side by side)."""
     decode_graph_safe = True
@@ -77,6 +85,10 @@ class PairRopeAttention(Mixer):
                 out.append(TensorSpec(p + "v.b", (G * V,), init="bias"))
         if spec.get("head_norm") == "weight":
             out += [TensorSpec(p + "q.norm", (D,), init="norm"), TensorSpec(p + "k.norm", (D,), init="norm")]
+        if spec.get("proj_norm"):
+            out += [TensorSpec(p + "q.norm", (H * D,), init="norm"), TensorSpec(p + "k.norm", (G * D,), init="norm")]
+        if spec.get("v_mix"):
+            out.append(TensorSpec(p + "vmix", (), init="fraction"))
         if spec.get("head_temp"):
             out.append(TensorSpec(p + "temp", (H,), init="norm"))
         if spec.get("sink_learned"):
@@ -84,6 +96,11 @@ class PairRopeAttention(Mixer):
         if spec.get("dist_bias"):
             out.append(TensorSpec(p + "rel", (int(spec["dist_bias"][0]), H), init="bias"))
         return out
+
+    @staticmethod
+    def _whole_rows(spec: PartSpec) -> bool:
+        """Whether a row's q, k and v are prepared together by one block (`ops.qk_norm_store`)."""
+        return bool(spec.get("proj_norm") or spec.get("v_mix") or spec.get("rot_layout", "pairs") != "pairs")
 
     @classmethod
     def cache_need(cls, spec: PartSpec):
@@ -93,7 +110,7 @@ class PairRopeAttention(Mixer):
 
     @classmethod
     def libraries(cls, spec, dtype):
-        out = [("rope_pairs", {})]
+        out = [("norm_attention" if cls._whole_rows(spec) else "rope_pairs", {})]
         head = ops.padded_head(spec["dim"], spec["vdim"])
         if dtype == torch.bfloat16 and ops.attention_tc_supported(head):
             out.append(("attention_tc", {"LAB_HEAD_DIM": head}))
@@ -120,17 +137,19 @@ class PairRopeAttention(Mixer):
         self.rot_dims = int(spec.get("rot_dims", self.dim))
         if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
             raise ValueError("pair_rope_attention: rot_dims must be even and at most dim")
-        i = np.arange(self.rot_dims // 2, dtype=np.float64)
-        inv = np.power(float(spec.get("rot_base") or 1.0), -2.0 * i / max(self.rot_dims, 1))
-        inv = (inv / float(spec.get("rot_scaling") or 1.0)).astype(np.float32)
-        self.inv_freq = torch.from_numpy(inv).to(device)
+        self.inv_freq = torch.from_numpy(rope_frequencies(spec.get("rot_base") or 1.0, self.rot_dims,
+                                                          spec.get("rot_scaling") or 1.0,
+                                                          spec.get("rot_bands"))).to(device)
+        if spec.get("rot_layout", "pairs") not in ("pairs", "halves"):
+            raise ValueError(f"pair_rope_attention: rot_layout {spec.get('rot_layout')!r} is not one of 'pairs', 'halves'")
         # the options that take the kernel with a norm per head and temperatures
         self.head_norm = spec.get("head_norm")
         if self.head_norm not in (None, "unit", "weight"):
             raise ValueError(f"pair_rope_attention: head_norm {self.head_norm!r} is not one of 'unit', 'weight'")
         self.eps = float(spec.get("eps") or 0.0)
-        if self.head_norm and not self.eps > 0.0:
-            raise ValueError("pair_rope_attention: a norm per head needs eps")
+        self.proj_norm = bool(spec.get("proj_norm"))
+        if (self.head_norm or self.proj_norm) and not self.eps > 0.0:
+            raise ValueError("pair_rope_attention: a norm of q and k needs eps")
         f32 = lambda n: weights[spec.prefix + n].to(device=device, dtype=torch.float32).contiguous()  # noqa: E731
         self.head_temp = f32("temp") if spec.get("head_temp") else None
         self.q_temp = tuple(spec["q_temp"]) if spec.get("q_temp") else None
@@ -143,12 +162,20 @@ class PairRopeAttention(Mixer):
             rel = f32("rel")
             self.dist_bias = distance_table(rel, rows if rows > 0 else rel.shape[0], far)     # -1: as many as stored
         self.prep = bool(self.head_norm or self.head_temp is not None or self.q_temp is not None)
+        self.v_mix = spec.get("v_mix") or None
+        if self.v_mix not in (None, "first", "mix"):
+            raise ValueError(f"pair_rope_attention: v_mix {self.v_mix!r} is not one of 'first', 'mix'")
+        self.lam = float(weights[spec.prefix + "vmix"]) if self.v_mix == "mix" else 0.0
+        self.whole_rows = self._whole_rows(spec)
+        if self.whole_rows and (self.prep or self.from_keys):
+            raise ValueError("pair_rope_attention: whole-projection norms, halves and mixed values go with neither a norm "
+                             "per head nor temperatures nor values taken from the keys")
         w = lambda n: self._weight(weights, n)  # noqa: E731
         names = ("q", "k") if self.from_keys else ("q", "k", "v")
         self.w_in = torch.cat([w(n) for n in names], dim=0).contiguous()
         self.bias_in = torch.cat([w(n + ".b") for n in names], dim=0).contiguous() if spec.get("bias") else None
-        self.norm_q = w("q.norm") if self.head_norm == "weight" else None
-        self.norm_k = w("k.norm") if self.head_norm == "weight" else None
+        self.norm_q = w("q.norm") if self.head_norm == "weight" or self.proj_norm else None
+        self.norm_k = w("k.norm") if self.head_norm == "weight" or self.proj_norm else None
         self.k_at = self.n_q * self.dim
         self.v_at = self.k_at if self.from_keys else self.k_at + self.n_kv * self.dim
         # the heads' outputs come `head` wide: zero columns of W_o meet the padding
@@ -169,7 +196,9 @@ class PairRopeAttention(Mixer):
             proj = ops.linear(x, self.w_in, None, out_f32=True, allow_partial=True)
         write = cache.write
         slots = group.row_slot if write else None
-        if self.prep:
+        if self.whole_rows:
+            q = self._prepare_rows(proj, ctx, slots, cache)
+        elif self.prep:
             coef, every = self.q_temp if self.q_temp is not None else (0.0, 0)
             q = ops.head_prep_store(proj, self.bias_in, ctx.row_pos, self.inv_freq, self.rot_dims, slots, cache.k,
                                     cache.v, self.n_q, self.n_kv, self.dim, self.vdim, self.head, self.k_at, self.v_at,
@@ -183,6 +212,22 @@ class PairRopeAttention(Mixer):
         return ops.attention(q, cache.k, cache.v, ctx, group, self.n_q, self.n_kv, self.head, self.window, self.scale,
                              keep_first=self.keep_first, sink_one=self.sink_one, sink=self.sink,
                              dist_bias=self.dist_bias)
+
+    def _prepare_rows(self, proj, ctx: StepContext, slots, cache: CacheView):
+        keep = first = None
+        if self.v_mix == "first":
+            keep = ctx.scratch["v_first"] = torch.empty((proj.shape[-2], self.n_kv * self.vdim), dtype=torch.float32,
+                                                        device=proj.device)
+        elif self.v_mix == "mix":
+            first = ctx.scratch.get("v_first")
+            if first is None:
+                raise ValueError("pair_rope_attention: no layer before this one has left its values")
+        write = slots is not None
+        return ops.qk_norm_store(proj, self.bias_in, self.norm_q, self.norm_k, slots, cache.k if write else None,
+                                 cache.v if write else None, self.n_q, self.n_kv, self.dim, self.vdim, self.head,
+                                 self.eps, dtype=self.dtype, positions=ctx.row_pos, inv_freq=self.inv_freq,
+                                 rot_dims=self.rot_dims, rot_pairs=self.spec.get("rot_layout", "pairs") == "pairs",
+                                 v_keep=keep, v_first=first, v_mix=self.lam)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
         attn = self.forward_inner(x, ctx, cache)

@@ -74,6 +74,8 @@ def _register_builtin() -> None:
     register_architecture("Bukatar", BukatarConfig, bukatar_blueprint)
     from .config.kupedra import KupedraConfig, kupedra_blueprint
     register_architecture("Kupedra", KupedraConfig, kupedra_blueprint)
+    from .config.difedra import DifedraConfig, difedra_blueprint
+    register_architecture("Difedra", DifedraConfig, difedra_blueprint)
 
 
 _register_builtin()
