@@ -1158,6 +1158,144 @@ def run_arch_kupedra(args):
     return 0
 
 
+# ----------------------------------------------------------------------------------------
+# --arch difedra: the Difedra design beside Bukatar and Qwen2 at equal layer sizes (random weights)
+# ----------------------------------------------------------------------------------------
+DIFEDRA_SHAPES = {
+    # width, vocabulary, attention heads and dense feed-forward of the Qwen2.5 shape of the same name; windows and
+    # experts as in the Bukatar shape of the same name
+    "0.5B": dict(heads=14, kv_heads=2, dim=64, vdim=64, window=512, experts=8, top=2, expert_ff=1536),
+    "1.5B": dict(heads=12, kv_heads=2, dim=128, vdim=128, window=1024, experts=8, top=2, expert_ff=2816),
+}
+
+
+def difedra_config(shape, layers):
+    """Windowed attention with mixed values in every layer; dense and routed feed-forwards alternate."""
+    q, m = SHAPES[shape], DIFEDRA_SHAPES[shape]
+    D = m["dim"]
+    mixer = {"heads": m["heads"], "kv_heads": m["kv_heads"], "dim": D, "vdim": m["vdim"], "scale": D ** -0.5, "v_mix": True,
+             "mask": {"size": m["window"]},
+             "rot": {"base": 500000.0, "dims": D, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    ffs = [{"kind": "dense", "ff": q["intermediate_size"]},
+           {"kind": "moe", "router": {"experts": m["experts"], "top": m["top"]}, "expert": {"ff": m["expert_ff"]}}]
+    return {"architecture": "Difedra", "vocab": q["vocab_size"], "width": q["hidden_size"], "norm": {"eps": 1e-6},
+            "max_positions": 4096, "layers": [{"type": "attention", "mixer": mixer, "mlp": ffs[i % 2]} for i in range(layers)]}
+
+
+def kernel_points_difedra(shape, batch, ctx_len, prefill_tokens, pk):
+    """The Difedra design's own kernels beside the like kernels of Bukatar (the attention's store, the windowed
+    attention, the sum that closes a sublayer, the experts' steps), of Ritizen (whole-projection norms) and of Qwen2
+    (the gated product) at the shape's sizes, each alone between CUDA events with L2 flushed: milliseconds and the
+    fraction of the roofline (measured copy bandwidth for kernels that stream, measured bf16 product rate for the
+    attention kernels and the products of a prompt)."""
+    import torch
+    from llm_inference_lab_b200.kernels import ops
+
+    dev = torch.device("cuda:0")
+    q, m = SHAPES[shape], DIFEDRA_SHAPES[shape]
+    width, ff = q["hidden_size"], q["intermediate_size"]
+    flush = torch.zeros((160 << 20,), dtype=torch.int16, device=dev)
+    bw, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    rows = {}
+
+    def record(name, ms, nbytes=None, flops=None):
+        entry = {"ms": round(ms, 4)}
+        if nbytes is not None:
+            entry.update(gbs=round(nbytes / (ms / 1e3) / 1e9, 1), frac_hbm=round(nbytes / (ms / 1e3) / bw, 4))
+        if flops is not None:
+            entry.update(tflops=round(flops / (ms / 1e3) / 1e12, 2), frac_bf16=round(flops / (ms / 1e3) / tf, 4))
+        rows[name] = entry
+
+    bf = lambda *s: (0.5 * torch.randn(*s, device=dev)).to(torch.bfloat16)  # noqa: E731
+    f32 = lambda *s: 0.5 * torch.randn(*s, device=dev)  # noqa: E731
+    nq, nkv, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    hd = ops.padded_head(D, V)
+    for label, q_lens, pos0 in (("prefill", [prefill_tokens], [0]), ("decode", [1] * batch, [ctx_len] * batch)):
+        T, B = sum(q_lens), len(q_lens)
+        ctx, pages = bench_ctx(q_lens, pos0, PAGE_SIZE, dev)
+        slots = ctx.groups[0].row_slot
+        # ---- whole-projection norms, rotation of halves, mixed values and the paged store, beside Ritizen's norms
+        # with the store and Bukatar's rotation with the store
+        ck, cv = bf(pages, nkv, PAGE_SIZE, hd), bf(pages, nkv, PAGE_SIZE, hd)
+        aproj, wq, wk = f32(T, nq * D + nkv * (D + V)), bf(nq * D), bf(nkv * D)
+        inv, first = torch.rand(D // 2, device=dev), f32(T, nkv * V)
+        io = T * ((nq * D + nkv * (D + V)) * 4 + (nq + 2 * nkv) * hd * 2)
+        for name, kw, extra in (
+                ("norms + rotation + mixed values", dict(positions=ctx.row_pos, inv_freq=inv, rot_dims=D, v_first=first, v_mix=0.4),
+                 T * nkv * V * 4),
+                ("norms + rotation, values left", dict(positions=ctx.row_pos, inv_freq=inv, rot_dims=D, v_keep=first),
+                 T * nkv * V * 4),
+                ("norms (ritizen)", {}, 0)):
+            ms = timed(lambda: ops.qk_norm_store(aproj, None, wq, wk, slots, ck, cv, nq, nkv, D, V, hd, 1e-6, **kw), flush=flush)
+            record(f"qk_norm_store {name} {label}", ms, nbytes=io + extra)
+        ms = timed(lambda: ops.rope_pairs_store(aproj, None, ctx.row_pos, inv, D, slots, ck, cv, nq, nkv, D, V, hd, nq * D,
+                                                (nq + nkv) * D, torch.bfloat16), flush=flush)
+        record(f"bukatar rope_pairs_store {label}", ms, nbytes=io)
+        # ---- attention: a window with learned sinks, beside the window with kept first tokens and the extra one
+        qq, sinks, win = bf(T, nq * hd), f32(nq), m["window"]
+        pairs = sum(sum(min(p + i + 1, win) for i in range(n)) for p, n in zip(pos0, q_lens))
+        keys = sum(min(p + n, win + n - 1) for p, n in zip(pos0, q_lens))
+        for name, kw in (("window + learned sink", dict(sink=sinks)), ("window + kept + one (bukatar)",
+                                                                       dict(sink_one=True, keep_first=4))):
+            ms = timed(lambda: ops.attention(qq, ck, cv, ctx, ctx.groups[0], nq, nkv, hd, win, D ** -0.5, **kw), flush=flush)
+            record(f"attention {name} {label}", ms, nbytes=keys * 2 * nkv * hd * 2 + 2 * T * nq * hd * 2,
+                   flops=4.0 * pairs * nq * hd)
+        # ---- the sum that closes a sublayer with the norm that opens the next one
+        one = torch.ones((1,), device=dev)
+        X, y, w1 = f32(T, 1, width), f32(T, width), bf(width)
+        ms = timed(lambda: ops.hyper_write(X, y, one.view(1, 1), one, one, w1, 1e-6), flush=flush)
+        record(f"residual sum + next norm {label}", ms, nbytes=T * width * (4 + 4 + 4 + 2))
+        ms = timed(lambda: ops.stream_norm_add(X.view(T, width), y, w1, 1e-6, next_weight=w1), flush=flush)
+        record(f"bukatar stream_norm_add + next norm {label}", ms, nbytes=T * width * (4 + 4 + 4 + 2))
+        # ---- the dense feed-forward: the GELU gate in the product's epilogue beside the SiLU gate
+        xb, w_gu = bf(T, width), bf(2 * ff, width)
+        for name, act in (("GELU", "gelu_tanh"), ("qwen2 SiLU", "silu")):
+            ms = timed(lambda: ops.linear_gated(xb, w_gu, act=act), flush=flush)
+            record(f"gated product, {name} gate {label}", ms, nbytes=(2 * ff * width + T * (width + ff)) * 2,
+                   flops=4.0 * T * ff * width)
+        # ---- the experts: sigmoid scores on the inputs beside softmax scores on the outputs
+        E, top, F = m["experts"], m["top"], m["expert_ff"]
+        logits = f32(T, E)
+        used = min(E, T * top)
+        w_egu, w_ed = bf(E, 2 * F, width), bf(E, width, F)
+        for name, score, renorm in (("sigmoid", "sigmoid", False), ("softmax (bukatar)", "softmax", True)):
+            ms = timed(lambda: ops.moe_route(logits, E, top, renorm=renorm, score=score), flush=flush)
+            record(f"moe_route, {name} {label}", ms, nbytes=T * (E * 4 + top * 8))
+        chosen, weight, _ = ops.moe_route(logits, E, top, renorm=False, score="sigmoid")
+        lay = ops.moe_layout(chosen, E, torch.bfloat16, width, F)
+        for name, scale in (("scaled inputs", weight), ("bukatar", None)):
+            ms = timed(lambda: ops.moe_experts_up(xb, w_egu, lay, top, in_scale=scale), flush=flush)
+            record(f"grouped gated product, {name} {label}", ms,
+                   nbytes=(used * 2 * F * width + T * width + T * top * F) * 2, flops=4.0 * T * top * F * width)
+        y2 = ops.moe_experts_down(ops.moe_experts_up(xb, w_egu, lay, top, in_scale=weight), w_ed, lay)
+        for name, w in (("plain sum", None), ("weighted sum (bukatar)", weight)):
+            ms = timed(lambda: ops.moe_combine(y2, lay.pos_of, w, None, None, top=top), flush=flush)
+            record(f"moe_combine, {name} {label}", ms, nbytes=T * width * 4 * (top + 1))
+    ops.take_device_errors()
+    return rows
+
+
+def run_arch_difedra(args):
+    shape, layers = args.shape, args.layers or 4
+    pk, pk_src = peaks()
+    qcfg = dict(SHAPES[shape], num_hidden_layers=layers)
+    folders = {"difedra": arch_folder(difedra_config(shape, layers), f"difedra_{shape}_L{layers}"),
+               "bukatar": arch_folder(bukatar_config(shape, layers), f"bukatar_{shape}_L{layers}"),
+               "qwen2": model_folder(SHAPES[shape], layers)}
+    clocks = ClockSampler()
+    with clocks:
+        models = {name: model_points(folder, args.batch, args.prompt_len, PREFILL_TOKENS, 20)
+                  for name, folder in folders.items()}
+        kernels = kernel_points_difedra(shape, args.batch, args.prompt_len + 512, PREFILL_TOKENS, pk)
+    print(json.dumps({
+        "arch": "difedra", "beside": ["bukatar", "qwen2"], "shape": shape, "layers": layers, "batch": args.batch,
+        "prompt_len": args.prompt_len, "prefill_tokens": PREFILL_TOKENS, "dtype": "bf16",
+        "data": "synthetic: random weights N(0, 0.02) seed 0", "difedra_mixers": DIFEDRA_SHAPES[shape],
+        "hidden": qcfg["hidden_size"], "intermediate": qcfg["intermediate_size"], "vocab": qcfg["vocab_size"],
+        "models": models, "kernels": kernels, "peaks": dict(pk, source=pk_src), "clocks": clocks.summary()}))
+    return 0
+
+
 def kv_bytes_per_token(cfg, layers):
     d = cfg["hidden_size"] // cfg["num_attention_heads"]
     return 2 * layers * 2 * cfg["num_key_value_heads"] * d
@@ -1186,12 +1324,13 @@ def main() -> int:
     ap.add_argument("--stack-stamps", action="store_true",
                     help="run a few eager decode steps with the decode stack's in-kernel clock on and print what "
                          "each kind of phase took")
-    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "sogulix", "ritizen", "bukatar", "kupedra"],
+    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "sogulix", "ritizen", "bukatar", "kupedra", "difedra"],
                     help="sogulix: instead of the headline run, prefill and decode throughput of the Sogulix design "
                          "beside Qwen2 at the layer sizes of --shape (0.5B or 1.5B; --layers, default 4), and each "
                          "of its kernels beside Qwen2's like kernel; prints its own line.  ritizen: the same for the "
                          "Ritizen design, beside Sogulix and Qwen2; bukatar: the same for the Bukatar design, beside "
-                         "Ritizen and Qwen2; kupedra: the same for the Kupedra design, beside Bukatar and Qwen2")
+                         "Ritizen and Qwen2; kupedra and difedra: the same for those "
+                         "designs, beside Bukatar and Qwen2")
     ap.add_argument("--only-prefill", type=int, default=0, metavar="TOKENS",
                     help="run only a prefill of TOKENS tokens a few times and print its time (for profiling)")
     args = ap.parse_args()
@@ -1238,6 +1377,11 @@ def main() -> int:
             ap.error("--arch kupedra knows the shapes " + ", ".join(sorted(KUPEDRA_SHAPES)))
         args.layers = 0 if args.layers == cfg["num_hidden_layers"] else args.layers
         return run_arch_kupedra(args)
+    if args.arch == "difedra":
+        if args.shape not in DIFEDRA_SHAPES:
+            ap.error("--arch difedra knows the shapes " + ", ".join(sorted(DIFEDRA_SHAPES)))
+        args.layers = 0 if args.layers == cfg["num_hidden_layers"] else args.layers
+        return run_arch_difedra(args)
     folder = model_folder(cfg, args.layers)
     pk, pk_src = peaks()
     if args.serve:

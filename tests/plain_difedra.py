@@ -152,10 +152,15 @@ def gated_mlp(h, w, p, act):
     return (act(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
-def routed_experts(h, w, p, mlp):
-    """Sigmoid scores; the chosen scores as they are multiply the experts' inputs."""
+def routed_experts(h, w, p, mlp, margins=None):
+    """Sigmoid scores; the chosen scores as they are multiply the experts' inputs.  `margins` (a list) receives, per
+    token, how far the last chosen expert's logit lies above the first one left out."""
     E, top = mlp["router"]["experts"], mlp["router"]["top"]
-    s = sigmoid(h @ w[p + "router"].T)
+    z = h @ w[p + "router"].T
+    s = sigmoid(z)
+    if margins is not None:
+        z = -np.sort(-z, axis=1)
+        margins.append(z[:, top - 1] - z[:, top] if top < E else np.full(len(z), np.inf))
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e in sorted(range(E), key=lambda e: (-s[t, e], e))[:top]:
@@ -166,8 +171,9 @@ def routed_experts(h, w, p, mlp):
 # ---------------------------------------------------------------------------------------------
 # the model
 # ---------------------------------------------------------------------------------------------
-def forward(cfg, w, tokens, layers_out=None):
-    """Logits [tokens, vocab] of one sequence; `layers_out` (a list) receives the residual after every layer."""
+def forward(cfg, w, tokens, layers_out=None, margins=None):
+    """Logits [tokens, vocab] of one sequence; `layers_out` (a list) receives the residual after every layer,
+    `margins` the routers' margins of every routed layer."""
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)]
     v_first = None
@@ -179,7 +185,7 @@ def forward(cfg, w, tokens, layers_out=None):
         if mlp is not None:
             h = rms_norm(x, w[p + "norm2"], eps)
             x = x + (gated_mlp(h, w, p + "mlp.", gelu_tanh) if mlp["kind"] == "dense"
-                     else routed_experts(h, w, p + "mlp.", mlp))
+                     else routed_experts(h, w, p + "mlp.", mlp, margins))
         if layers_out is not None:
             layers_out.append(x)
     return rms_norm(x, w["final.norm"], eps) @ w["embed"].T
