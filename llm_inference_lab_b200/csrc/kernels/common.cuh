@@ -139,6 +139,53 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return t;
 }
 
+// Two sums over a block at once; `scratch` holds 64 floats.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  __syncthreads();
+  if (lane == 0) {
+    scratch[warp] = a;
+    scratch[32 + warp] = b;
+  }
+  __syncthreads();
+  float2 t = lane < nwarps ? make_float2(scratch[lane], scratch[32 + lane]) : make_float2(0.f, 0.f);
+  t.x = warp_sum(t.x);
+  t.y = warp_sum(t.y);
+  return t;
+}
+
+// ---- four neighbours at a time (addresses on 16-byte, of bfloat16 8-byte, boundaries) -------
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(q.x << 16), __uint_as_float(q.x & 0xffff0000u), __uint_as_float(q.y << 16),
+                     __uint_as_float(q.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+// four entries of `splits` partial products `stride` floats apart, summed in ascending order, eight loads in flight
+__device__ __forceinline__ float4 sum_splits4(const float* __restrict__ p, int splits, long long stride, size_t at) {
+  if (splits == 1) return load4(p + at);
+  float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s0 = 0; s0 < splits; s0 += 8) {
+    float4 v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = s0 + j < splits ? load4(p + (s0 + j) * stride + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      t.x += v[j].x;
+      t.y += v[j].y;
+      t.z += v[j].z;
+      t.w += v[j].w;
+    }
+  }
+  return t;
+}
+
 #define LAB_LAUNCH_CHECK() return (int)cudaGetLastError()
 
 // ---- programmatic dependent launch --------------------------------------------------------

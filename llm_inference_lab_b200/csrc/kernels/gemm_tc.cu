@@ -510,9 +510,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
               uint32_t ru[32];
               tmem_ld32_issue(lane_addr + BN / 2 + c * 32, ru);
               tmem_wait();
-#pragma unroll
-              for (int j = 0; j < 32; ++j)
-                v[j] = gate_value(__uint_as_float(r[j]) * scale, __uint_as_float(ru[j]) * scale, p.gate_act, p.gate_limit);
+              if (p.row_scale != nullptr) gate_columns<true>(v, r, ru, p.gate_act, p.gate_limit, scale);
+              else gate_columns<false>(v, r, ru, p.gate_act, p.gate_limit, 1.f);
             } else {
               tmem_wait();
 #pragma unroll

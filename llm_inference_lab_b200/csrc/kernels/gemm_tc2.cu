@@ -262,9 +262,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc2_kernel(const __grid_constant
             uint32_t ru[32];
             tmem_ld32_issue(lane_addr + BN / 2 + c * 32, ru);
             tmem_wait();
-#pragma unroll
-            for (int j = 0; j < 32; ++j)
-              v[j] = gate_value(__uint_as_float(r[j]), __uint_as_float(ru[j]), p.gate_act, p.gate_limit);
+            gate_columns<false>(v, r, ru, p.gate_act, p.gate_limit, 1.f);
           } else {
             tmem_wait();
 #pragma unroll

@@ -183,6 +183,128 @@ __global__ void __launch_bounds__(kThreads) scale_rows_kernel(float* __restrict_
     x[i] *= c;
 }
 
+// ---- rows of whole groups of four: four coordinates a thread and load, all of a thread's loads in flight before the
+// first sum, the row kept in registers between the sum of squares and the norm.  U groups a thread.
+__device__ __forceinline__ float4 fma4(float c, float4 a, float4 b) {
+  return make_float4(fmaf(c, a.x, b.x), fmaf(c, a.y, b.y), fmaf(c, a.z, b.z), fmaf(c, a.w, b.w));
+}
+
+template <typename T>
+__device__ __forceinline__ float4 weight4_at(const T* __restrict__ w, int scalar, int i) {
+  if (!scalar) return load4(w + i);
+  const float v = to_f32(w[0]);
+  return make_float4(v, v, v, v);
+}
+
+template <typename T>
+__device__ __forceinline__ void store_normed4(T* dst, float4 u, float inv, float4 w) {
+  store4(dst, make_float4(u.x * inv * w.x, u.y * inv * w.y, u.z * inv * w.z, u.w * inv * w.w));
+}
+
+template <typename T, int THREADS, int U>
+__global__ void __launch_bounds__(THREADS) hyper_read_norm_vec_kernel(T* __restrict__ out, const float* __restrict__ X,
+                                                                      const float* __restrict__ c_in,
+                                                                      const T* __restrict__ w, int w_scalar,
+                                                                      const int* __restrict__ rows, int n_in, int S,
+                                                                      int hidden, float eps) {
+  __shared__ float scratch[32];
+  pdl_trigger();
+  pdl_wait();
+  int t = blockIdx.x;
+  if (rows != nullptr) {
+    t = rows[blockIdx.x];
+    if (t < 0 || t >= n_in) {
+      if (threadIdx.x == 0) lab_set_error(LAB_ERR_ROW_RANGE);
+      t = min(max(t, 0), n_in - 1);
+    }
+  }
+  const float* x = X + (size_t)t * S * hidden;
+  const int n4 = hidden / 4;
+  float4 u[U];
+#pragma unroll
+  for (int k = 0; k < U; ++k) u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s = 0; s < S; ++s) {
+    const float c = c_in != nullptr ? c_in[s] : 1.f;
+#pragma unroll
+    for (int k = 0; k < U; ++k) {
+      const int g = threadIdx.x + k * THREADS;
+      if (g < n4) u[k] = fma4(c, load4(x + (size_t)s * hidden + 4 * g), u[k]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < U; ++k) ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+#pragma unroll
+  for (int k = 0; k < U; ++k) {
+    const int g = threadIdx.x + k * THREADS;
+    if (g < n4) store_normed4(out + (size_t)blockIdx.x * hidden + 4 * g, u[k], inv, weight4_at(w, w_scalar, 4 * g));
+  }
+}
+
+template <typename T, int SMAX, int THREADS, int U>
+__global__ void __launch_bounds__(THREADS) hyper_write_vec_kernel(float* __restrict__ X, T* __restrict__ out,
+                                                                  const float* __restrict__ y, int y_splits,
+                                                                  long long split_stride, const float* __restrict__ mix,
+                                                                  const float* __restrict__ c_out,
+                                                                  const float* __restrict__ c_in_next,
+                                                                  const T* __restrict__ w_next, int w_scalar, int S,
+                                                                  int hidden, float eps) {
+  __shared__ float scratch[32];
+  __shared__ HyperCoef coef;
+  pdl_trigger();
+  for (int i = threadIdx.x; i < S * S; i += THREADS) coef.mix[i] = mix[i];
+  for (int i = threadIdx.x; i < S; i += THREADS) {
+    coef.c_out[i] = c_out[i];
+    coef.c_in[i] = c_in_next != nullptr ? c_in_next[i] : 0.f;
+  }
+  pdl_wait();
+  __syncthreads();
+  const int t = blockIdx.x, n4 = hidden / 4;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float* x = X + (size_t)t * S * hidden;
+  float4 old[U][SMAX], yv[U];
+#pragma unroll
+  for (int k = 0; k < U; ++k) {
+    const int g = threadIdx.x + k * THREADS;
+#pragma unroll
+    for (int s = 0; s < SMAX; ++s) old[k][s] = g < n4 && s < S ? load4(x + (size_t)s * hidden + 4 * g) : zero;
+    yv[k] = g < n4 ? sum_splits4(y, y_splits, split_stride, (size_t)t * hidden + 4 * g) : zero;
+  }
+  float4 u[U];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < U; ++k) {
+    const int g = threadIdx.x + k * THREADS;
+    u[k] = zero;
+#pragma unroll
+    for (int r = 0; r < SMAX; ++r) {
+      if (r >= S) break;
+      float4 v = zero;
+#pragma unroll
+      for (int s = 0; s < SMAX; ++s)
+        if (s < S) v = fma4(coef.mix[s * S + r], old[k][s], v);
+      v = fma4(coef.c_out[r], yv[k], v);
+      if (g < n4) store4(x + (size_t)r * hidden + 4 * g, v);
+      u[k] = fma4(coef.c_in[r], v, u[k]);
+    }
+    ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;
+  }
+  if (out == nullptr) return;
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+#pragma unroll
+  for (int k = 0; k < U; ++k) {
+    const int g = threadIdx.x + k * THREADS;
+    if (g < n4) store_normed4(out + (size_t)t * hidden + 4 * g, u[k], inv, weight4_at(w_next, w_scalar, 4 * g));
+  }
+}
+
+bool on16(const void* p) { return (((uintptr_t)p) & 15) == 0; }
+// rows the vector kernels take: whole groups of four, at most two groups a thread of 512
+bool rows_of_fours(int hidden) { return hidden % 4 == 0 && hidden / 4 <= 1024; }
+
 template <typename K>
 void allow_smem(K kernel, size_t smem) {
   if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -193,6 +315,18 @@ int launch_write(float* X, void* out, const float* y, int y_splits, const float*
                  const float* c_in_next, const void* w_next, int w_scalar, int tokens, int S, int hidden, float eps,
                  cudaStream_t stream) {
   const size_t smem = (size_t)hidden * sizeof(float);
+  if (SMAX <= 4 && rows_of_fours(hidden) && on16(X) && on16(y) && on16(out) && (w_scalar || on16(w_next))) {
+    constexpr int SV = SMAX <= 4 ? SMAX : 4;
+    auto run = [&](auto kernel, int threads) {
+      return (int)lab_launch(kernel, dim3(tokens), dim3(threads), 0, stream, X, (T*)out, y, y_splits,
+                             (long long)tokens * hidden, mix, c_out, c_in_next, (const T*)w_next, w_scalar, S, hidden, eps);
+    };
+    const int n4 = hidden / 4;
+    if (n4 <= 128) return run(hyper_write_vec_kernel<T, SV, 128, 1>, 128);
+    if (n4 <= 256) return run(hyper_write_vec_kernel<T, SV, 128, 2>, 128);
+    if (n4 <= 512) return run(hyper_write_vec_kernel<T, SV, 256, 2>, 256);
+    return run(hyper_write_vec_kernel<T, SV, 512, 2>, 512);
+  }
   allow_smem(hyper_write_kernel<T, SMAX>, smem);
   return (int)lab_launch(hyper_write_kernel<T, SMAX>, dim3(tokens), dim3(kThreads), smem, stream, X, (T*)out, y, y_splits,
                          (long long)tokens * hidden, mix, c_out, c_in_next, (const T*)w_next, w_scalar, S, hidden, eps);
@@ -202,12 +336,34 @@ template <typename T>
 int launch_write_for(int S, float* X, void* out, const float* y, int y_splits, const float* mix, const float* c_out,
                      const float* c_in_next, const void* w_next, int w_scalar, int tokens, int hidden, float eps,
                      cudaStream_t stream) {
+  if (S == 1)
+    return launch_write<T, 1>(X, out, y, y_splits, mix, c_out, c_in_next, w_next, w_scalar, tokens, S, hidden, eps, stream);
   if (S <= 2)
     return launch_write<T, 2>(X, out, y, y_splits, mix, c_out, c_in_next, w_next, w_scalar, tokens, S, hidden, eps, stream);
   if (S <= 4)
     return launch_write<T, 4>(X, out, y, y_splits, mix, c_out, c_in_next, w_next, w_scalar, tokens, S, hidden, eps, stream);
   return launch_write<T, kMaxStreams>(X, out, y, y_splits, mix, c_out, c_in_next, w_next, w_scalar, tokens, S, hidden, eps,
                                       stream);
+}
+
+template <typename T>
+int launch_read_norm(void* out, const float* X, const float* c_in, const void* w, int w_scalar, const int* rows, int n_out,
+                     int n_in, int S, int hidden, float eps, cudaStream_t stream) {
+  if (rows_of_fours(hidden) && on16(X) && on16(out) && (w_scalar || on16(w))) {
+    auto run = [&](auto kernel, int threads) {
+      return (int)lab_launch(kernel, dim3(n_out), dim3(threads), 0, stream, (T*)out, X, c_in, (const T*)w, w_scalar, rows,
+                             n_in, S, hidden, eps);
+    };
+    const int n4 = hidden / 4;
+    if (n4 <= 128) return run(hyper_read_norm_vec_kernel<T, 128, 1>, 128);
+    if (n4 <= 256) return run(hyper_read_norm_vec_kernel<T, 128, 2>, 128);
+    if (n4 <= 512) return run(hyper_read_norm_vec_kernel<T, 256, 2>, 256);
+    return run(hyper_read_norm_vec_kernel<T, 512, 2>, 512);
+  }
+  const size_t smem = (size_t)hidden * sizeof(float);
+  allow_smem(hyper_read_norm_kernel<T>, smem);
+  return (int)lab_launch(hyper_read_norm_kernel<T>, dim3(n_out), dim3(kThreads), smem, stream, (T*)out, X, c_in, (const T*)w,
+                         w_scalar, rows, n_in, S, hidden, eps);
 }
 }  // namespace
 
@@ -226,16 +382,8 @@ LAB_EXPORT int lab_hyper_read_norm(void* out, const float* X, const float* c_in,
   if (n_out <= 0) return 0;
   const size_t smem = (size_t)hidden * sizeof(float);
   if (S < 1 || S > kMaxStreams || smem > 200 * 1024) return (int)cudaErrorInvalidValue;
-  if (dtype == LAB_F32) {
-    allow_smem(hyper_read_norm_kernel<float>, smem);
-    lab_launch(hyper_read_norm_kernel<float>, dim3(n_out), dim3(kThreads), smem, stream, (float*)out, X, c_in,
-               (const float*)w, w_scalar, rows, n_in, S, hidden, eps);
-  } else {
-    allow_smem(hyper_read_norm_kernel<__nv_bfloat16>, smem);
-    lab_launch(hyper_read_norm_kernel<__nv_bfloat16>, dim3(n_out), dim3(kThreads), smem, stream, (__nv_bfloat16*)out, X,
-               c_in, (const __nv_bfloat16*)w, w_scalar, rows, n_in, S, hidden, eps);
-  }
-  LAB_LAUNCH_CHECK();
+  if (dtype == LAB_F32) return launch_read_norm<float>(out, X, c_in, w, w_scalar, rows, n_out, n_in, S, hidden, eps, stream);
+  return launch_read_norm<__nv_bfloat16>(out, X, c_in, w, w_scalar, rows, n_out, n_in, S, hidden, eps, stream);
 }
 
 // out / c_in_next / w_next null: the write alone.

@@ -150,16 +150,33 @@ __global__ void __launch_bounds__(kThreads) moe_combine_kernel(float* __restrict
                                                                const float* __restrict__ weight,
                                                                const float* __restrict__ shared,
                                                                const float* __restrict__ shared_gate, int top,
-                                                               int width) {
+                                                               int width, int vec) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
+  const int* pos = pos_of + (size_t)t * top;
+  const float* wt = weight != nullptr ? weight + (size_t)t * top : nullptr;
+  if (vec) {      // rows of whole groups of four
+    const float gs = shared != nullptr ? (shared_gate != nullptr ? shared_gate[t] : 1.f) : 0.f;
+    for (int i = 4 * threadIdx.x; i < width; i += 4 * kThreads) {
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+      auto add = [&](float c, float4 v) {
+        acc = make_float4(fmaf(c, v.x, acc.x), fmaf(c, v.y, acc.y), fmaf(c, v.z, acc.z), fmaf(c, v.w, acc.w));
+      };
+#pragma unroll 2
+      for (int k = 0; k < top; ++k)
+        if (pos[k] >= 0) add(wt != nullptr ? wt[k] : 1.f, load4(y + (size_t)pos[k] * width + i));
+      if (shared != nullptr) add(gs, load4(shared + (size_t)t * width + i));
+      store4(out + (size_t)t * width + i, acc);
+    }
+    return;
+  }
   const float g = shared != nullptr ? (shared_gate != nullptr ? shared_gate[t] : 1.f) : 0.f;
   for (int i = threadIdx.x; i < width; i += kThreads) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
-      const int at = pos_of[(size_t)t * top + k];
-      if (at >= 0) acc = fmaf(weight != nullptr ? weight[(size_t)t * top + k] : 1.f, y[(size_t)at * width + i], acc);
+      const int at = pos[k];
+      if (at >= 0) acc = fmaf(wt != nullptr ? wt[k] : 1.f, y[(size_t)at * width + i], acc);
     }
     if (shared != nullptr) acc = fmaf(g, shared[(size_t)t * width + i], acc);
     out[(size_t)t * width + i] = acc;
@@ -204,7 +221,8 @@ LAB_EXPORT int lab_moe_gather(void* out, const void* x, const int* row_src, int 
 LAB_EXPORT int lab_moe_combine(float* out, const float* y, const int* pos_of, const float* weight, const float* shared,
                                const float* shared_gate, int tokens, int top, int width, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  const int vec = width % 4 == 0 && ((((uintptr_t)out) | ((uintptr_t)y) | ((uintptr_t)shared)) & 15) == 0;
   lab_launch(moe_combine_kernel, dim3(tokens), dim3(kThreads), 0, stream, out, y, pos_of, weight, shared, shared_gate, top,
-             width);
+             width, vec);
   LAB_LAUNCH_CHECK();
 }

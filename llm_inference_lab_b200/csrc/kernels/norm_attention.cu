@@ -129,6 +129,141 @@ __global__ void __launch_bounds__(kThreads) qk_norm_store_kernel(T* __restrict__
   }
 }
 
+// the same on four entries i .. i + 3 of a head: all of one half (or whole pairs), the mates likewise side by side
+template <typename T>
+__device__ __forceinline__ float4 normed_rotated4(const float* h, const T* w, float inv, int i, const QkNormParams& p,
+                                                  const float* cs, const float* sn) {
+  auto normed = [&](int at) {
+    float4 a = load4(h + at);
+    if (w != nullptr) {
+      const float4 g = load4(w + at);
+      a.x = a.x * inv * g.x; a.y = a.y * inv * g.y; a.z = a.z * inv * g.z; a.w = a.w * inv * g.w;
+    }
+    return a;
+  };
+  float4 a = normed(i), r;
+  if (i >= 2 * p.rot_half) return a;
+  if (p.rot_pairs) {
+    const int f = i >> 1;
+    rope_rotate(a.x, a.y, cs[f], sn[f], r.x, r.y);
+    rope_rotate(a.z, a.w, cs[f + 1], sn[f + 1], r.z, r.w);
+    return r;
+  }
+  const bool low = i < p.rot_half;
+  const int f = low ? i : i - p.rot_half;
+  const float4 b = normed(low ? i + p.rot_half : f), c = load4(cs + f), s = load4(sn + f);
+  const float4 lo = low ? a : b, hi = low ? b : a;
+  float4 ol, oh;
+  rope_rotate(lo.x, hi.x, c.x, s.x, ol.x, oh.x);
+  rope_rotate(lo.y, hi.y, c.y, s.y, ol.y, oh.y);
+  rope_rotate(lo.z, hi.z, c.z, s.z, ol.z, oh.z);
+  rope_rotate(lo.w, hi.w, c.w, s.w, ol.w, oh.w);
+  return low ? ol : oh;
+}
+
+// qk_norm_store for sizes that are whole groups of four (head sizes, row stride, the rotated half): four entries a
+// thread and load, two loads a thread in flight before anything is summed, the angles formed while they arrive, and
+// both root mean squares from one block-wide sum.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) qk_norm_store_vec_kernel(T* __restrict__ q_out, T* __restrict__ cache_k,
+                                                                     T* __restrict__ cache_v,
+                                                                     const T* __restrict__ bias,
+                                                                     const T* __restrict__ wq, const T* __restrict__ wk,
+                                                                     QkNormParams p) {
+  extern __shared__ __align__(16) float row[];      // as above
+  __shared__ float scratch[64];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int wq_n = p.n_q * p.D, wk_n = p.has_kv ? p.n_kv * p.D : 0, wv_n = p.has_kv ? p.n_kv * p.V : 0;
+  const int n4 = (wq_n + wk_n + wv_n) / 4;
+  float *cs = row + 4 * n4, *sn = cs + p.rot_half;
+  const int slot = p.has_kv && cache_k != nullptr ? p.slots[t] : -1;
+  float ssq = 0.f, ssk = 0.f;
+  bool angles = p.rot_half > 0;
+  for (int g0 = threadIdx.x; g0 < n4; g0 += 2 * kThreads) {
+    float4 v[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int g = g0 + j * kThreads;
+      v[j] = g < n4 ? sum_splits4(p.proj, p.splits, p.split_stride, (size_t)t * p.ld + 4 * g) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (angles) {
+      angles = false;
+      const float pos = (float)p.positions[t];
+      for (int i = threadIdx.x; i < p.rot_half; i += kThreads) sincosf(pos * p.inv_freq[i], &sn[i], &cs[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = 4 * (g0 + j * kThreads);
+      if (i >= 4 * n4) break;
+      float4 a = v[j];
+      if (bias != nullptr) {
+        const float4 b = load4(bias + i);
+        a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
+      }
+      const float ss = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+      if (i < wq_n) {
+        ssq += ss;
+      } else if (i < wq_n + wk_n) {
+        ssk += ss;
+      } else {
+        const size_t at = (size_t)t * wv_n + i - wq_n - wk_n;
+        if (p.v_keep != nullptr) store4(p.v_keep + at, a);
+        if (p.v_first != nullptr) {
+          const float4 f = load4(p.v_first + at);
+          const float m = p.v_mix, o = 1.f - p.v_mix;
+          a = make_float4(o * a.x + m * f.x, o * a.y + m * f.y, o * a.z + m * f.z, o * a.w + m * f.w);
+        }
+      }
+      store4(row + i, a);
+    }
+  }
+  if (angles) {      // threads without an entry of the row may have an angle to form
+    const float pos = (float)p.positions[t];
+    for (int i = threadIdx.x; i < p.rot_half; i += kThreads) sincosf(pos * p.inv_freq[i], &sn[i], &cs[i]);
+  }
+  const float2 ss = block_sum2(ssq, ssk, scratch);
+  const float inv_q = 1.0f / sqrtf(ss.x / (float)wq_n + p.eps);
+  const int per = p.HD / 4;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int g = threadIdx.x; g < p.n_q * per; g += kThreads) {
+    const int h = g / per, i = 4 * (g - h * per);
+    store4(q_out + (size_t)t * p.ld_q + 4 * g,
+           i < p.D ? normed_rotated4(row + h * p.D, wq != nullptr ? wq + h * p.D : nullptr, inv_q, i, p, cs, sn) : zero);
+  }
+  if (slot == -1) return;
+  const int page = slot / p.page_size, off = slot - page * p.page_size;
+  if (slot < 0 || page >= p.num_pages) {
+    if (threadIdx.x == 0) lab_set_error(LAB_ERR_PAGE_RANGE);
+    return;
+  }
+  const float inv_k = 1.0f / sqrtf(ss.y / (float)wk_n + p.eps);
+  // the last threads first: they are the ones with fewest of q's groups
+  for (int g = kThreads - 1 - threadIdx.x; g < 2 * p.n_kv * per; g += kThreads) {
+    const bool is_v = g >= p.n_kv * per;
+    const int e = is_v ? g - p.n_kv * per : g, h = e / per, i = 4 * (e - h * per);
+    T* dst = (is_v ? cache_v : cache_k) + (((size_t)page * p.n_kv + h) * p.page_size + off) * p.HD + i;
+    if (is_v) store4(dst, i < p.V ? load4(row + wq_n + wk_n + h * p.V + i) : zero);
+    else store4(dst, i < p.D ? normed_rotated4(row + wq_n + h * p.D, wk != nullptr ? wk + h * p.D : nullptr, inv_k, i, p, cs, sn)
+                             : zero);
+  }
+}
+
+template <typename T>
+int launch_qk_norm_store(void* q_out, void* cache_k, void* cache_v, const void* bias, const void* wq, const void* wk,
+                         const QkNormParams& p, int tokens, size_t smem, cudaStream_t stream) {
+  auto on16 = [](const void* a) { return (((uintptr_t)a) & 15) == 0; };
+  const bool vec = p.D % 4 == 0 && p.V % 4 == 0 && p.HD % 4 == 0 && p.ld % 4 == 0 && p.split_stride % 4 == 0 &&
+                   p.ld_q % 4 == 0 && p.rot_half % (p.rot_pairs ? 2 : 4) == 0 && on16(p.proj) && on16(q_out) && on16(cache_k) &&
+                   on16(cache_v) && on16(bias) && on16(wq) && on16(wk) && on16(p.v_keep) && on16(p.v_first);
+  auto kernel = vec ? qk_norm_store_vec_kernel<T> : qk_norm_store_kernel<T>;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  lab_launch(kernel, dim3(tokens), dim3(kThreads), smem, stream, (T*)q_out, (T*)cache_k, (T*)cache_v, (const T*)bias,
+             (const T*)wq, (const T*)wk, p);
+  LAB_LAUNCH_CHECK();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kThreads) head_gate_kernel(T* __restrict__ out, int ld_o, const T* __restrict__ attn,
                                                              int ld_a, const float* __restrict__ proj, int splits,
@@ -172,19 +307,8 @@ LAB_EXPORT int lab_qk_norm_store(void* q_out, int ld_q, void* cache_k, void* cac
   p.rot_half = rot_dims / 2; p.rot_pairs = rot_pairs; p.v_keep = v_keep; p.v_first = v_first; p.v_mix = v_mix;
   const size_t smem = (size_t)(n_q * D + (has_kv ? n_kv * (D + V) : 0) + rot_dims) * sizeof(float);
   if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
-  if (dtype == LAB_F32) {
-    if (smem > 48 * 1024)
-      cudaFuncSetAttribute(qk_norm_store_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    lab_launch(qk_norm_store_kernel<float>, dim3(tokens), dim3(kThreads), smem, stream, (float*)q_out, (float*)cache_k,
-               (float*)cache_v, (const float*)bias, (const float*)wq, (const float*)wk, p);
-  } else {
-    if (smem > 48 * 1024)
-      cudaFuncSetAttribute(qk_norm_store_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    lab_launch(qk_norm_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(kThreads), smem, stream, (__nv_bfloat16*)q_out,
-               (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v, (const __nv_bfloat16*)bias, (const __nv_bfloat16*)wq,
-               (const __nv_bfloat16*)wk, p);
-  }
-  LAB_LAUNCH_CHECK();
+  if (dtype == LAB_F32) return launch_qk_norm_store<float>(q_out, cache_k, cache_v, bias, wq, wk, p, tokens, smem, stream);
+  return launch_qk_norm_store<__nv_bfloat16>(q_out, cache_k, cache_v, bias, wq, wk, p, tokens, smem, stream);
 }
 
 // attn: [tokens, ld_a] of T with heads HD wide; the gate's pre-activations start at column gate_at of proj.

@@ -193,24 +193,40 @@ __host__ __device__ constexpr uint32_t umma_instr_desc(int m, int n, bool b_n_ma
 // fewer roundings only come closer to the exact value); exp and the division use the hardware
 // approximations (relative error about 2^-21, far below bfloat16's 2^-9).
 __device__ __forceinline__ float silu_gate(float g, float u) { return __fdividef(g, 1.f + __expf(-g)) * u; }
-// The same with the capped form of the gate (`gate_pair` in common.cuh): a positive limit caps g from above and
-// u on both sides, the sigmoid reads 1.702 g and u enters as u + 1; limit 0 is silu(g) * u.
-__device__ __forceinline__ float silu_gate(float g, float u, float limit) {
-  if (limit > 0.f) {
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
-  }
-  return silu_gate(g, u);
+// The same with the capped form of the gate (`gate_pair` in common.cuh): `limit` caps g from above and u on both
+// sides, the sigmoid reads 1.702 g and u enters as u + 1.
+__device__ __forceinline__ float capped_gate(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
 }
-// The same by the gate's activation: 1, the tanh form of GELU of g, times u, with 0.5 (1 + tanh(y)) written as the
-// sigmoid of 2 y; 0, as above.
+// The tanh form of GELU of g, times u: 0.5 (1 + tanh(y)) is the sigmoid of 2 y, y = sqrt(2/pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float gelu_gate(float g, float u) {
+  const float twice = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+  return __fdividef(g, 1.f + __expf(-twice)) * u;
+}
+// By the gate's activation: 1, GELU; 0, SiLU with limit 0 and the capped form with a positive one.
 __device__ __forceinline__ float gate_value(float g, float u, int act, float limit) {
-  if (act == 1) {
-    const float twice = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
-    return __fdividef(g, 1.f + __expf(-twice)) * u;
+  if (act == 1) return gelu_gate(g, u);
+  return limit > 0.f ? capped_gate(g, u, limit) : silu_gate(g, u);
+}
+// 32 accumulator columns of gate (r) and up (ru) to their gated values, every pair multiplied by `scale` first where
+// SCALED.  The kind of gate is decided once for all of them.
+template <bool SCALED>
+__device__ __forceinline__ void gate_columns(float (&v)[32], const uint32_t (&r)[32], const uint32_t (&ru)[32], int act,
+                                             float limit, float scale) {
+  auto g = [&](int j) { return SCALED ? __uint_as_float(r[j]) * scale : __uint_as_float(r[j]); };
+  auto u = [&](int j) { return SCALED ? __uint_as_float(ru[j]) * scale : __uint_as_float(ru[j]); };
+  if (act == 0 && !(limit > 0.f)) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = silu_gate(g(j), u(j));
+  } else if (act == 0) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = capped_gate(g(j), u(j), limit);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = gelu_gate(g(j), u(j));
   }
-  return silu_gate(g, u, limit);
 }
 
 // ---- host: tensor maps -----------------------------------------------------------------------

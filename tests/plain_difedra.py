@@ -138,7 +138,7 @@ def attention(h, w, p, m, eps, v_first):
         if v_first is None:
             v_first = v
         else:
-            v = mixed_values(v, v_first, float(w[p + "vmix"]))
+            v = mixed_values(v, v_first, float(np.reshape(w[p + "vmix"], -1)[0]))
     v = v.reshape(T, G, V)
     per = H // G
     s = np.stack([q[:, i] @ k[:, i // per].T for i in range(H)]) * m["scale"]

@@ -54,7 +54,7 @@ def _rotate(v, positions, freq, pairs):
 @pytest.mark.parametrize("H,G,D,V,dims,pairs,norm", [
     (4, 2, 16, 24, 8, False, True), (3, 3, 40, 8, 40, False, True), (1, 1, 12, 20, 2, False, True),
     (5, 1, 24, 24, 24, True, True), (2, 2, 32, 16, 16, False, False), (6, 3, 10, 130, 0, False, True),
-    (8, 1, 128, 64, 96, False, True)])
+    (8, 1, 128, 64, 96, False, True), (3, 1, 16, 8, 2, True, True), (14, 2, 96, 64, 96, True, True), (2, 2, 8, 12, 4, False, True)])
 def test_whole_projection_norms_rotation_and_mixed_values(H, G, D, V, dims, pairs, norm):
     """q and k normed over all heads at once and then rotated (halves, or neighbours), the values left for later
     layers and mixed with those an earlier layer left, everything stored in the rows' slots with zeros beyond a
@@ -71,7 +71,7 @@ def test_whole_projection_norms_rotation_and_mixed_values(H, G, D, V, dims, pair
     pos = ctx.row_pos.cpu().numpy()
     width = H * D + G * (D + V)
     for dtype in _dtypes():
-        tol = 2e-5 if dtype == torch.float32 else 0.04
+        tol = 4e-5 if dtype == torch.float32 else 0.04      # an angle of 130 radians, rounded, is 8e-6 off
         wq, wk = (_t(1 + 0.3 * rng.standard_normal(n * D), dtype) if norm else None for n in (H, G))
         for splits in (1, 3):
             proj = _t(rng.standard_normal((splits, T, width)))
