@@ -62,13 +62,15 @@ __device__ __forceinline__ long long key_offset(const int* __restrict__ bt, int 
 //   before a window.  m, l, o carry the running max (log2 units), sum and accumulator.
 //   bias0 / bias1 (bias_len > 0): a table by distance for each of the thread's two rows, in natural units;
 //   entry min(hi[i] - j, bias_len - 1) is added to the scaled score (hi[i] is the row's own position).
+//   cap_log2 > 0: scores are capped first (`softcapped_log2` with arg_log2).
 template <int BN>
 __device__ __forceinline__ void tile_step(const uint32_t (&qf)[KSTEPS][4], uint32_t ks, uint32_t vs,
                                           float (&o)[DTILES][4], float (&m)[2], float (&l)[2], int key0,
                                           const int (&lo)[2], const int (&hi)[2], float scale_log2, int lane,
                                           bool all_visible = false, int keep = 0,
                                           const float* __restrict__ bias0 = nullptr,
-                                          const float* __restrict__ bias1 = nullptr, int bias_len = 0) {
+                                          const float* __restrict__ bias1 = nullptr, int bias_len = 0,
+                                          float cap_log2 = 0.f, float arg_log2 = 0.f) {
   float s[BN / 8][4];
 #pragma unroll
   for (int j = 0; j < BN / 8; ++j)
@@ -86,6 +88,13 @@ __device__ __forceinline__ void tile_step(const uint32_t (&qf)[KSTEPS][4], uint3
       mma_bf16(s[2 * jp], qf[k], b[0], b[1]);
       mma_bf16(s[2 * jp + 1], qf[k], b[2], b[3]);
     }
+  }
+  if (cap_log2 > 0.f) {
+#pragma unroll
+    for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[j][e] = softcapped_log2(s[j][e], arg_log2, cap_log2);
+    scale_log2 = 1.f;      // in log2 units already
   }
   // mask, scale, running max
   float mx[2] = {-INFINITY, -INFINITY};

@@ -17,7 +17,8 @@
 // that many positions stay visible to every later query, at their true positions) and `sink` (1: one is
 // added to the softmax's denominator, a key with score 0 and no value; with `sinks`, a number per query head,
 // exp(sinks[h]) instead), and `dist_bias` [n_q, bias_len]: a number per head and distance query - key that is
-// added to the scaled score, distances from bias_len - 1 on sharing the last entry.
+// added to the scaled score, distances from bias_len - 1 on sharing the last entry.  `softcap` c > 0: the scaled score
+// s becomes c * tanh(s / c) first.
 #include "common.cuh"
 
 namespace {
@@ -30,7 +31,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_plain_kernel(
     const T* __restrict__ cache_v, const int* __restrict__ row_req, const int* __restrict__ row_pos,
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int d, int page_size, int num_pages,
     int window, float scale, int keep_first, int sink, const float* __restrict__ sinks,
-    const float* __restrict__ dist_bias, int bias_len) {
+    const float* __restrict__ dist_bias, int bias_len, float softcap) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
@@ -69,6 +70,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_plain_kernel(
         float dot = 0.f;
         for (int i = 0; i < d; ++i) dot = fmaf(qs[i], to_f32<T>(kr[i]), dot);
         s = dot * scale;
+        if (softcap > 0.f) s = softcap * tanhf(s / softcap);
         if (dist_bias != nullptr) s += dist_bias[(size_t)h * bias_len + min(p - j, bias_len - 1)];
       }
     }
@@ -126,7 +128,8 @@ LAB_EXPORT int lab_attention_plain(void* out, int out_stride, const void* q, int
                                    const void* cache_v, const int* row_req, const int* row_pos, const int* block_table,
                                    int max_blocks, int tokens, int n_q, int n_kv, int d, int page_size, int num_pages,
                                    int window, float scale, int keep_first, int sink, const float* sinks,
-                                   const float* dist_bias, int bias_len, int dtype, cudaStream_t stream) {
+                                   const float* dist_bias, int bias_len, float softcap, int dtype,
+                                   cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (d > 32 * MAX_DPL || d <= 0 || n_q % n_kv || (dist_bias != nullptr && bias_len < 1)) return (int)cudaErrorInvalidValue;
   if (sinks != nullptr) sink = 1;
@@ -136,10 +139,10 @@ LAB_EXPORT int lab_attention_plain(void* out, int out_stride, const void* q, int
     return (int)lab_launch(attention_plain_kernel<float>, grid, dim3(WARPS * 32), smem, stream, (float*)out, out_stride,
                            (const float*)q, q_stride, (const float*)cache_k, (const float*)cache_v, row_req, row_pos,
                            block_table, max_blocks, n_q, n_kv, d, page_size, num_pages, window, scale, keep_first,
-                           sink, sinks, dist_bias, bias_len);
+                           sink, sinks, dist_bias, bias_len, softcap);
   return (int)lab_launch(attention_plain_kernel<__nv_bfloat16>, grid, dim3(WARPS * 32), smem, stream,
                          (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
                          (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v, row_req, row_pos, block_table,
                          max_blocks, n_q, n_kv, d, page_size, num_pages, window, scale, keep_first, sink, sinks, dist_bias,
-                         bias_len);
+                         bias_len, softcap);
 }

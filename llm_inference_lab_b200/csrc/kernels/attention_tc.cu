@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(PF_THREADS) attention_prefill_kernel(
     const int* __restrict__ q_start, const int* __restrict__ kv_len_arr, const int* __restrict__ pos0_arr,
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window,
     float scale_log2, int min_q_len, const float* __restrict__ sink, int keep, const float* __restrict__ dist_bias,
-    int bias_len) {
+    int bias_len, float cap_log2, float arg_log2) {
   extern __shared__ __align__(16) uint8_t smem[];
   pdl_trigger();
   pdl_wait();
@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(PF_THREADS) attention_prefill_kernel(
                                (window == 0 || t * PF_BN >= lab_first_key(p0 + first_row + 15, window) ||
                                 t * PF_BN + PF_BN <= keep);
       tile_step<PF_BN>(qf, kd, kd + PF_TILE_BYTES, o, m, l, t * PF_BN, lo, hi, scale_log2, lane, all_visible, keep,
-                       bias_h, bias_h, bias_len);
+                       bias_h, bias_h, bias_len, cap_log2, arg_log2);
     }
     __syncthreads();  // the stage is refilled by the next iteration's prefetch
   }
@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
     const int* __restrict__ q_start, const int* __restrict__ kv_len_arr, const int* __restrict__ block_table,
     int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window, float scale_log2, int splits,
     float* __restrict__ part_acc, float* __restrict__ part_ml, int keep, const float* __restrict__ sink,
-    const float* __restrict__ dist_bias, int bias_len) {
+    const float* __restrict__ dist_bias, int bias_len, float cap_log2, float arg_log2) {
   extern __shared__ __align__(16) uint8_t smem[];
   using L = DcLayout<CLUSTER>;
   pdl_trigger();
@@ -314,7 +314,7 @@ __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
     // every key of an inner tile is visible to the one query row: no mask to evaluate
     tile_step<DC_BN>(qf, kd, kd + DC_TILE_BYTES, o, m, l, key0, lo, hi, scale_log2, lane,
                      (key0 >= first || key0 + DC_BN <= keep) && key0 + DC_BN <= kvl, keep, bias_r[0], bias_r[1],
-                     bias_len);
+                     bias_len, cap_log2, arg_log2);
     __syncwarp();
     stage = (stage + 1) % L::STAGES;
   }
@@ -458,12 +458,17 @@ LAB_EXPORT long long lab_attention_decode_scratch_floats(int requests, int n_q, 
   return splits > 1 ? (long long)requests * n_q * splits * (D + 2) : 0;
 }
 
+// the kernels' two numbers of a soft cap (0: none)
+static float cap_of(float softcap) { return softcap > 0.f ? softcap * LOG2E : 0.f; }
+static float cap_arg(float softcap, float scale) { return softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f; }
+
+// softcap c > 0: the scaled score s becomes c * tanh(s / c), before a bias by distance.
 LAB_EXPORT int lab_attention_prefill(void* out, int out_stride, const void* q, int q_stride, const void* cache_k,
                                      const void* cache_v, const int* q_start, const int* kv_len, const int* pos0,
                                      const int* block_table, int max_blocks, int requests, int max_q_len, int n_q,
                                      int n_kv, int page_size, int num_pages, int window, float scale, int min_q_len,
                                      const float* sink, int keep_first, const float* dist_bias, int bias_len,
-                                     cudaStream_t stream) {
+                                     float softcap, cudaStream_t stream) {
   if (requests <= 0 || max_q_len <= 0) return 0;
   if (n_q % n_kv || q_stride % 8 || (((uintptr_t)q) & 15)) return (int)cudaErrorInvalidValue;
   static bool configured = false;
@@ -477,7 +482,8 @@ LAB_EXPORT int lab_attention_prefill(void* out, int out_stride, const void* q, i
                          (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
                          (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v, q_start, kv_len, pos0,
                          block_table, max_blocks, n_q, n_kv, page_size, num_pages, window, scale * LOG2E, min_q_len,
-                         sink, window > 0 && keep_first > 0 ? keep_first : 0, dist_bias, dist_bias != nullptr ? bias_len : 0);
+                         sink, window > 0 && keep_first > 0 ? keep_first : 0, dist_bias, dist_bias != nullptr ? bias_len : 0,
+                         cap_of(softcap), cap_arg(softcap, scale));
 }
 
 static int decode_launch(void* out, int out_stride, const void* q, int q_stride, const void* cache_k,
@@ -485,7 +491,7 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
                          int max_blocks, int requests, int n_q, int n_kv, int page_size, int num_pages, int window,
                          float scale, int splits, float* scratch, bool may_cluster, cudaStream_t stream,
                          int keep_first = 0, const float* sink = nullptr, const float* dist_bias = nullptr,
-                         int bias_len = 0) {
+                         int bias_len = 0, float softcap = 0.f) {
   if (requests <= 0) return 0;
   if (dist_bias == nullptr) bias_len = 0;
   const int keep = window > 0 && keep_first > 0 ? keep_first : 0;
@@ -525,7 +531,7 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
                                    (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v,
                                    q_start, kv_len, block_table, max_blocks, n_q, n_kv, page_size, num_pages, window,
                                    scale * LOG2E, splits, (float*)nullptr, (float*)nullptr, keep, sink, dist_bias,
-                                   bias_len);
+                                   bias_len, cap_of(softcap), cap_arg(softcap, scale));
   }
   float* part_acc = scratch;
   float* part_ml = scratch ? scratch + (size_t)requests * n_q * splits * D : nullptr;
@@ -533,7 +539,7 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
                              (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
                              (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v, q_start, kv_len, block_table,
                              max_blocks, n_q, n_kv, page_size, num_pages, window, scale * LOG2E, splits, part_acc,
-                             part_ml, keep, sink, dist_bias, bias_len);
+                             part_ml, keep, sink, dist_bias, bias_len, cap_of(softcap), cap_arg(softcap, scale));
   if (e != cudaSuccess) return (int)e;
   if (splits > 1)
     e = lab_launch(attention_merge_kernel, dim3(requests, n_q), dim3(D), 0, stream, (__nv_bfloat16*)out, out_stride,
@@ -547,16 +553,16 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
 // keep_first: beside a window, the first that many positions stay visible; sink: null or a number per
 // query head that joins the softmax's denominator as exp(sink); dist_bias: null or [n_q, bias_len] floats, a
 // number per head and distance query - key added to the scaled score (distances from bias_len - 1 on share the
-// last entry).
+// last entry); softcap: as lab_attention_prefill.
 LAB_EXPORT int lab_attention_decode(void* out, int out_stride, const void* q, int q_stride, const void* cache_k,
                                     const void* cache_v, const int* q_start, const int* kv_len,
                                     const int* block_table, int max_blocks, int requests, int n_q, int n_kv,
                                     int page_size, int num_pages, int window, float scale, int splits, float* scratch,
                                     int cluster_merge, int keep_first, const float* sink, const float* dist_bias,
-                                    int bias_len, cudaStream_t stream) {
+                                    int bias_len, float softcap, cudaStream_t stream) {
   return decode_launch(out, out_stride, q, q_stride, cache_k, cache_v, q_start, kv_len, block_table, max_blocks,
                        requests, n_q, n_kv, page_size, num_pages, window, scale, splits, scratch, cluster_merge != 0,
-                       stream, keep_first, sink, dist_bias, bias_len);
+                       stream, keep_first, sink, dist_bias, bias_len, softcap);
 }
 
 // ----------------------------------------------------------------------------------------

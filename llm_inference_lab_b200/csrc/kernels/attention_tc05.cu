@@ -87,7 +87,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc05_kernel(
     const int* __restrict__ q_start, const int* __restrict__ kv_len_arr, const int* __restrict__ pos0_arr,
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window,
     float scale_log2, int min_q_len, int keep, const float* __restrict__ sink, const float* __restrict__ dist_bias,
-    int bias_len, float bias_mult) {
+    int bias_len, float bias_mult, float cap_log2, float arg_log2) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   Barriers* bar = reinterpret_cast<Barriers*>(smem + OFF_BAR);
@@ -325,6 +325,10 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc05_kernel(
         for (int c = 0; c < BN / 32; ++c) tmem_ld32_issue(lane_addr + TM_S + sb * BN + c * 32, sr + c * 32);
         tmem_wait();
         const int key0 = tile_of(j) * BN;
+        if (cap_log2 > 0.f) {      // the scores leave in log2 units (scale_log2 is 1 then)
+#pragma unroll
+          for (int c = 0; c < BN; ++c) sr[c] = __float_as_uint(softcapped_log2(__uint_as_float(sr[c]), arg_log2, cap_log2));
+        }
         if (bias_len > 0) {
           const int d0 = pos - key0;      // the distance to the tile's first key; consecutive rows read consecutive entries
 #pragma unroll
@@ -457,14 +461,15 @@ LAB_EXPORT int lab_attention_tc05_supports(int page_size) {
 // keep_first: beside a window, the first that many positions stay visible; sink: null or a number per
 // query head that joins the softmax's denominator as exp(sink); dist_bias: null or [n_q, bias_len] floats
 // (bias_len up to lab_attention_tc05_bias_max()), a number per head and distance query - key added to the scaled
-// score, distances from bias_len - 1 on sharing the last entry.
+// score, distances from bias_len - 1 on sharing the last entry.  softcap c > 0: the scaled score s becomes
+// c * tanh(s / c), before the bias.
 LAB_EXPORT int lab_attention_tc05_bias_max() { return BIAS_MAX; }
 LAB_EXPORT int lab_attention_prefill_tc05(void* out, int out_stride, const void* q, int q_stride, int total_rows,
                                           const void* cache_k, const void* cache_v, const int* q_start,
                                           const int* kv_len, const int* pos0, const int* block_table, int max_blocks,
                                           int requests, int max_q_len, int n_q, int n_kv, int page_size, int num_pages,
                                           int window, float scale, int min_q_len, int keep_first, const float* sink,
-                                          const float* dist_bias, int bias_len, cudaStream_t stream) {
+                                          const float* dist_bias, int bias_len, float softcap, cudaStream_t stream) {
   if (requests <= 0 || max_q_len <= 0) return 0;
   if (dist_bias == nullptr) bias_len = 0;
   if (bias_len < 0 || bias_len > BIAS_MAX || !(scale > 0.f)) return (int)cudaErrorInvalidValue;
@@ -488,6 +493,7 @@ LAB_EXPORT int lab_attention_prefill_tc05(void* out, int out_stride, const void*
   return (int)lab_launch(attention_prefill_tc05_kernel, grid, dim3(THREADS), (size_t)SMEM, stream, mq, mk, mv,
                          (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v,
                          q_start, kv_len, pos0, block_table, max_blocks, n_q, n_kv, page_size, num_pages, window,
-                         scale * LOG2E, min_q_len, window > 0 && keep_first > 0 ? keep_first : 0, sink, dist_bias, bias_len,
-                         1.0f / scale);
+                         softcap > 0.f ? 1.f : scale * LOG2E, min_q_len, window > 0 && keep_first > 0 ? keep_first : 0, sink,
+                         dist_bias, bias_len, softcap > 0.f ? LOG2E : 1.0f / scale, softcap > 0.f ? softcap * LOG2E : 0.f,
+                         softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f);
 }

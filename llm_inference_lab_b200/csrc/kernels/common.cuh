@@ -64,6 +64,12 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// A score under a soft cap: cap * tanh(raw * scale / cap) in log2 units, by the hardware's 2^x and reciprocal
+// approximations (absolute error about 2^-21 of the cap): tanh(y) = 1 - 2 / (1 + e^2y).  cap_log2 = cap * log2(e),
+// arg_log2 = 2 * log2(e) * scale / cap.
+__device__ __forceinline__ float softcapped_log2(float raw, float arg_log2, float cap_log2) {
+  return fmaf(-2.f * cap_log2, __fdividef(1.f, 1.f + fast_exp2(raw * arg_log2)), cap_log2);
+}
 // ---- thread-block clusters ---------------------------------------------------------------
 __device__ __forceinline__ uint32_t cluster_rank() {
   uint32_t r;

@@ -82,7 +82,13 @@ __global__ void __launch_bounds__(kThreads) rope_pairs_store_kernel(T* __restric
 // root) and multiplied by a weight of `dim` entries that all heads share (null: no weight); then q is
 // multiplied by a number per head (`q_head_scale`, null: 1) and by 1 + coef * ln(floor((pos + 1) / every) + 1)
 // (`every` 0: 1).  One warp per (row, head), a head's entries over the lanes.
+//
+// `maps` M > 1 (several score maps over the same values): n_q counts query heads and maps together, a key/value
+// head holds M keys of `dim` entries side by side (M * dim <= head), and query i, which belongs to map i % M, lies
+// at the entries of its map's key, zeros elsewhere, so that its product with the whole head meets that key alone.
+// `v_rep` R > 1: key head g is stored with the values of value head g / R.
 struct HeadPrepParams {
+  int maps, v_rep;
   float norm_eps;          // <= 0: no norm
   const float* q_head_scale;
   float temp_coef;
@@ -99,7 +105,7 @@ __global__ void __launch_bounds__(kThreads) head_prep_store_kernel(T* __restrict
   pdl_wait();
   constexpr int kPerLane = 8;      // heads of up to 256 entries
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int units = p.n_q + 2 * p.n_kv;
+  const int n_keys = p.n_kv * hp.maps, units = p.n_q + n_keys + p.n_kv;
   const long long unit = (long long)blockIdx.x * (kThreads / 32) + warp;
   if (unit >= (long long)tokens * units) return;
   const int t = (int)(unit / units), u = (int)(unit - (long long)t * units);
@@ -107,8 +113,9 @@ __global__ void __launch_bounds__(kThreads) head_prep_store_kernel(T* __restrict
   const int ipos = p.positions[t];
   const float pos = (float)ipos;
   const int HD = p.head;
-  const bool is_q = u < p.n_q, is_v = u >= p.n_q + p.n_kv;
-  const int g = is_q ? u : (is_v ? u - p.n_q - p.n_kv : u - p.n_q);
+  const bool is_q = u < p.n_q, is_v = u >= p.n_q + n_keys;
+  const int g = is_q ? u : (is_v ? u - p.n_q - n_keys : u - p.n_q);      // query, value head, or key (head and map)
+  const int map = is_v ? 0 : g % hp.maps, place = map * p.dim;             // where the vector lies in its head
   T* dst;
   if (is_q) {
     dst = q_out + ((size_t)t * p.n_q + g) * HD;
@@ -121,11 +128,13 @@ __global__ void __launch_bounds__(kThreads) head_prep_store_kernel(T* __restrict
       return;
     }
     const long long page = slot / p.page_size, off = slot % p.page_size;
-    dst = (is_v ? cache_v : cache_k) + (((size_t)page * p.n_kv + g) * p.page_size + off) * HD;
+    const int head = is_v ? g : g / hp.maps;
+    dst = (is_v ? cache_v : cache_k) + (((size_t)page * p.n_kv + head) * p.page_size + off) * HD;
   }
   if (is_v) {
+    const int col = p.v_at + (g / hp.v_rep) * p.vdim;
     for (int e = lane; e < HD; e += 32)
-      dst[e] = from_f32<T>(e < p.vdim ? rotated_entry(p, bias, row, p.v_at + g * p.vdim, e, pos, false) : 0.f);
+      dst[e] = from_f32<T>(e < p.vdim ? rotated_entry(p, bias, row, col, e, pos, false) : 0.f);
     return;
   }
   const int col = is_q ? g * p.dim : p.k_at + g * p.dim;
@@ -147,11 +156,14 @@ __global__ void __launch_bounds__(kThreads) head_prep_store_kernel(T* __restrict
 #pragma unroll
   for (int i = 0; i < kPerLane; ++i) {
     const int e = lane + 32 * i;
-    if (e >= HD) break;
+    if (e >= p.dim) break;
     float v = val[i] * mult;
-    if (w != nullptr && e < p.dim) v *= to_f32(w[e]);
-    dst[e] = from_f32<T>(v * after);
+    if (w != nullptr) v *= to_f32(w[e]);
+    dst[place + e] = from_f32<T>(v * after);
   }
+  // zeros: around a query, behind the last key of a head
+  for (int e = lane; e < HD; e += 32)
+    if (is_q ? (e < place || e >= place + p.dim) : (map == hp.maps - 1 && e >= place + p.dim)) dst[e] = from_f32<T>(0.f);
 }
 }  // namespace
 
@@ -179,25 +191,26 @@ LAB_EXPORT int lab_rope_pairs_store(void* q_out, void* cache_k, void* cache_v, c
 
 // As lab_rope_pairs_store, with the norm per head (norm_eps > 0; weights q_norm_w, k_norm_w of `dim` entries or
 // null) and q's temperatures (q_head_scale [n_q] floats or null; temp_every > 0: 1 + temp_coef * ln(floor((pos + 1)
-// / temp_every) + 1)).  rot_dims may be 0: no rotation.
+// / temp_every) + 1)).  rot_dims may be 0: no rotation.  maps, v_rep: see HeadPrepParams (1: neither); with v_rep > 1
+// the projection holds n_kv / v_rep value heads.
 LAB_EXPORT int lab_head_prep_store(void* q_out, void* cache_k, void* cache_v, const float* proj, int splits,
                                    long long split_stride, int ld, int k_at, int v_at, const void* bias,
                                    const int* positions, const float* inv_freq, int rot_dims, const int* slots,
                                    long long n_slots, int tokens, int n_q, int n_kv, int dim, int vdim, int head,
                                    int page_size, float norm_eps, const void* q_norm_w, const void* k_norm_w,
-                                   const float* q_head_scale, float temp_coef, int temp_every, int dtype,
-                                   cudaStream_t stream) {
+                                   const float* q_head_scale, float temp_coef, int temp_every, int maps, int v_rep,
+                                   int dtype, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || dim > head || vdim > head || splits < 1 || page_size < 1 ||
-      head > 256 || temp_every < 0)
+      dim > 256 || temp_every < 0 || maps < 1 || v_rep < 1 || maps * dim > head || n_q % maps || n_kv % v_rep)
     return (int)cudaErrorInvalidValue;
   RopePairsParams p;
   p.proj = proj; p.split_stride = split_stride; p.splits = splits; p.ld = ld; p.k_at = k_at; p.v_at = v_at;
   p.positions = positions; p.inv_freq = inv_freq; p.slots = slots; p.n_slots = n_slots; p.n_q = n_q; p.n_kv = n_kv;
   p.dim = dim; p.vdim = vdim; p.head = head; p.rot_dims = rot_dims; p.page_size = page_size;
   HeadPrepParams hp;
-  hp.norm_eps = norm_eps; hp.q_head_scale = q_head_scale; hp.temp_coef = temp_coef; hp.temp_every = temp_every;
-  const long long units = (long long)tokens * (n_q + 2 * n_kv);
+  hp.maps = maps; hp.v_rep = v_rep; hp.norm_eps = norm_eps; hp.q_head_scale = q_head_scale; hp.temp_coef = temp_coef; hp.temp_every = temp_every;
+  const long long units = (long long)tokens * (n_q + (maps + 1) * n_kv);
   const int blocks = (int)((units + kThreads / 32 - 1) / (kThreads / 32));
   if (dtype == LAB_F32)
     lab_launch(head_prep_store_kernel<float>, dim3(blocks), dim3(kThreads), 0, stream, (float*)q_out, (float*)cache_k,

@@ -1,7 +1,8 @@
 // Row-wise operators for models whose residual stream is kept in 32-bit floats whatever the
 // storage type T of weights and activations is: embedding with a norm, RMS norms that read the
 // 32-bit stream (one or two at once, gain w or 1 + w), embedding with a learned position, the sum
-// x += norm(product) of blocks that norm a sublayer's output, token shift with a per-request previous
+// x += norm(product) of blocks that norm a sublayer's output, x = norm(alpha x + product) of blocks that norm the
+// sum, a gate by a token's own vector, token shift with a per-request previous
 // row, the block's sum into the stream with per-channel scales (alone, or as the opening of the
 // next block's norms, as the 16-bit stream's add + norm kernel has it), concatenation for a re-entry
 // projection, and a soft cap on logits.  All arithmetic is 32-bit; T only says how weights are
@@ -256,6 +257,68 @@ __global__ void __launch_bounds__(1024) stream_norm_add_kernel(float* __restrict
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) copy[base + i] = from_f32<T>(row[i] * inv2 * to_f32(w_next[i]));
 }
 
+// ---- x = norm(alpha x + product): the sum that closes a sublayer of a block that norms the stream itself ----
+// v = alpha * x[t] + a[t], a a 32-bit product or split-K partial products summed in ascending order;
+// x[t] = v / rms(v) * w, and (if asked) the new x[t] rounded to T for the product that reads it next.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(1024) stream_post_norm_kernel(float* __restrict__ x, T* __restrict__ copy,
+                                                                const float* __restrict__ a, int a_splits,
+                                                                long long split_stride, const T* __restrict__ w,
+                                                                int hidden, float alpha, float eps) {
+  __shared__ float scratch[32];
+  extern __shared__ __align__(16) float row[];      // [hidden]: the sum
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const size_t base = (size_t)t * hidden;
+  float ss = 0.f;
+  if constexpr (VEC) {      // rows of whole groups of four
+    for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
+      const float4 p = sum_splits4(a, a_splits, split_stride, base + i), o = load4(x + base + i);
+      const float4 v = make_float4(fmaf(alpha, o.x, p.x), fmaf(alpha, o.y, p.y), fmaf(alpha, o.z, p.z), fmaf(alpha, o.w, p.w));
+      store4(row + i, v);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+      const float v = fmaf(alpha, x[base + i], sum_splits(a, a_splits, split_stride, base + i));
+      row[i] = v;
+      ss += v * v;
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+  if constexpr (VEC) {
+    for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
+      const float4 v = load4(row + i), g = load4(w + i);
+      const float4 y = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+      store4(x + base + i, y);
+      if (copy != nullptr) store4(copy + base + i, y);
+    }
+  } else {
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+      const float y = row[i] * inv * to_f32(w[i]);
+      x[base + i] = y;
+      if (copy != nullptr) copy[base + i] = from_f32<T>(y);
+    }
+  }
+}
+
+// ---- a product gated by the token's own vector: out = gelu(p) * table[id, at ...] -----------------
+// p [tokens, n] a 32-bit product or split-K partial products; the table's rows are `ld` wide.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) token_gate_kernel(T* __restrict__ out, const float* __restrict__ p, int splits,
+                                                              const T* __restrict__ table, const int* __restrict__ ids,
+                                                              long long total, int n, int ld, int at, int vocab) {
+  pdl_trigger();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * kThreads + threadIdx.x; i < total; i += (long long)gridDim.x * kThreads) {
+    const long long t = i / n;
+    const int c = (int)(i - t * n), id = min(max(ids[t], 0), vocab - 1);
+    out[i] = from_f32<T>(gelu_tanh_f(sum_splits(p, splits, total, (size_t)i)) * to_f32(table[(size_t)id * ld + at + c]));
+  }
+}
+
 // ---- the stream rounded to T ------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(kThreads) stream_round_kernel(T* __restrict__ out, const float* __restrict__ x,
@@ -441,5 +504,41 @@ LAB_EXPORT int lab_stream_concat(void* out, const float* x, const float* x0, lon
 LAB_EXPORT int lab_softcap(float* logits, long long n, float cap, cudaStream_t stream) {
   if (n <= 0) return 0;
   lab_launch(softcap_kernel, dim3(blocks_for(n)), dim3(kThreads), 0, stream, logits, n, cap);
+  LAB_LAUNCH_CHECK();
+}
+
+template <typename T>
+static int launch_post_norm(float* x, void* copy, const float* a, int a_splits, const void* w, int tokens, int hidden,
+                            float alpha, float eps, cudaStream_t stream) {
+  const size_t smem = (size_t)hidden * sizeof(float);
+  auto on16 = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
+  const bool vec = hidden % 4 == 0 && on16(x) && on16(copy) && on16(a) && on16(w);
+  auto kernel = vec ? stream_post_norm_kernel<T, true> : stream_post_norm_kernel<T, false>;
+  const int per = vec ? (hidden + 3) / 4 : hidden;
+  const int threads = tokens <= 64 || per < kThreads ? (per >= 1024 ? 1024 : (per + 31) / 32 * 32) : kThreads;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  return (int)lab_launch(kernel, dim3(tokens), dim3(threads), smem, stream, x, (T*)copy, a, a_splits,
+                         (long long)tokens * hidden, (const T*)w, hidden, alpha, eps);
+}
+
+LAB_EXPORT int lab_stream_post_norm(float* x, void* copy, const float* a, int a_splits, const void* w, int tokens,
+                                    int hidden, float alpha, float eps, int dtype, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (hidden <= 0 || (size_t)hidden * sizeof(float) > 160 * 1024) return (int)cudaErrorInvalidValue;
+  if (dtype == LAB_F32) return launch_post_norm<float>(x, copy, a, a_splits, w, tokens, hidden, alpha, eps, stream);
+  return launch_post_norm<__nv_bfloat16>(x, copy, a, a_splits, w, tokens, hidden, alpha, eps, stream);
+}
+
+LAB_EXPORT int lab_token_gate(void* out, const float* p, int splits, const void* table, const int* ids, long long tokens,
+                              int n, int ld, int at, int vocab, int dtype, cudaStream_t stream) {
+  const long long total = tokens * n;
+  if (total <= 0) return 0;
+  if (at < 0 || at + n > ld) return (int)cudaErrorInvalidValue;
+  if (dtype == LAB_F32)
+    lab_launch(token_gate_kernel<float>, dim3(blocks_for(total)), dim3(kThreads), 0, stream, (float*)out, p, splits,
+               (const float*)table, ids, total, n, ld, at, vocab);
+  else
+    lab_launch(token_gate_kernel<__nv_bfloat16>, dim3(blocks_for(total)), dim3(kThreads), 0, stream, (__nv_bfloat16*)out, p,
+               splits, (const __nv_bfloat16*)table, ids, total, n, ld, at, vocab);
   LAB_LAUNCH_CHECK();
 }

@@ -316,11 +316,12 @@ def attention_plain(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tenso
                     row_pos: torch.Tensor, block_table: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
                     window: int, scale: float, out: torch.Tensor | None = None, keep_first: int = 0,
                     sink_one: bool = False, sink: torch.Tensor | None = None,
-                    dist_bias: torch.Tensor | None = None) -> torch.Tensor:
+                    dist_bias: torch.Tensor | None = None, softcap: float = 0.0) -> torch.Tensor:
     """Attention of every row over its request's pages; q may be a column slice of the fused projection.
     `keep_first`: with a window, the first that many positions stay visible; `sink_one`: one more in the
     softmax's denominator; `sink` [n_q] 32-bit: exp(sink[h]) more instead; `dist_bias` [n_q, L] 32-bit: added to
-    the scaled score by distance query - key, distances from L - 1 on sharing the last entry."""
+    the scaled score by distance query - key, distances from L - 1 on sharing the last entry; `softcap` c > 0: the
+    scaled score s becomes c * tanh(s / c), before the bias."""
     _on_gpu(q, cache_k, cache_v, row_req, row_pos, block_table, sink, dist_bias)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() >= n_q and sink.is_contiguous())
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.dim() == 2 and
@@ -335,7 +336,8 @@ def attention_plain(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tenso
         _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(cache_k), _ptr(cache_v), _ptr(row_req), _ptr(row_pos),
         _ptr(block_table), block_table.shape[1], tokens, n_q, n_kv, head_dim, page_size, num_pages, window,
         ctypes.c_float(scale), int(keep_first), int(bool(sink_one) or sink is not None), _ptr(sink), _ptr(dist_bias),
-        dist_bias.shape[1] if dist_bias is not None else 0, dtype_code(q.dtype), _stream()), "attention_plain")
+        dist_bias.shape[1] if dist_bias is not None else 0, ctypes.c_float(softcap), dtype_code(q.dtype), _stream()),
+        "attention_plain")
     return out
 
 
@@ -739,14 +741,15 @@ TC05_BIAS_MAX = 4096     # entries of a distance table the tcgen05 prefill kerne
 
 def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requests, q_lens, max_kv_len,
                  n_q, n_kv, head_dim, window, scale, out=None, splits=None, scratch=None, keep_first=0, sink=None,
-                 dist_bias=None):
+                 dist_bias=None, softcap=0.0):
     """Tensor-core attention: the prefill kernel serves requests with several new tokens,
     the split-KV decode kernel those with one.  A negative `window` means chunks of that many positions.
     `keep_first`: beside a window, the first that many positions stay visible.  `sink`: 32-bit numbers, one per
     query head, that join the softmax's denominator as exp(sink) (a key with that unscaled score and no value).
     `dist_bias` [n_q, L] 32-bit: a number per head and distance query - key added to the scaled score, distances
     from L - 1 on sharing the last entry (the tcgen05 kernel keeps a head's table in shared memory, up to
-    `TC05_BIAS_MAX` entries; longer tables run on the `mma.sync` prefill kernel)."""
+    `TC05_BIAS_MAX` entries; longer tables run on the `mma.sync` prefill kernel).  `softcap` c > 0: the scaled score
+    s becomes c * tanh(s / c), before the bias."""
     _on_gpu(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, sink, dist_bias)
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.dim() == 2 and
                                  dist_bias.shape[0] == n_q and dist_bias.is_contiguous())
@@ -773,14 +776,14 @@ def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requ
             _ptr(out), out.stride(0), _ptr(q), q.stride(0), tokens, _ptr(cache_k), _ptr(cache_v), _ptr(q_start),
             _ptr(kv_len), _ptr(pos0), _ptr(block_table), block_table.shape[1], n_requests, max_q, n_q, n_kv,
             page_size, num_pages, window, ctypes.c_float(scale), 2, keep_first, _ptr(sink), _ptr(dist_bias), bias_len,
-            _stream()),
+            ctypes.c_float(softcap), _stream()),
             "attention_prefill_tc05")
     elif max_q > 1:
         _check(L.lab_attention_prefill(_ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(cache_k), _ptr(cache_v),
                                        _ptr(q_start), _ptr(kv_len), _ptr(pos0), _ptr(block_table),
                                        block_table.shape[1], n_requests, max_q, n_q, n_kv, page_size, num_pages,
                                        window, ctypes.c_float(scale), 2, _ptr(sink), keep_first, _ptr(dist_bias),
-                                       bias_len, _stream()),
+                                       bias_len, ctypes.c_float(softcap), _stream()),
                "attention_prefill")
     if n_decode:
         if splits is None:
@@ -798,21 +801,22 @@ def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requ
                                       _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.shape[1],
                                       n_requests, n_q, n_kv, page_size, num_pages, window, ctypes.c_float(scale),
                                       splits, _ptr(scratch), 1 if in_cluster else 0, keep_first, _ptr(sink),
-                                      _ptr(dist_bias), bias_len, _stream()),
+                                      _ptr(dist_bias), bias_len, ctypes.c_float(softcap), _stream()),
                "attention_decode",
                2 if splits > 1 and not in_cluster else 1)
     return out
 
 
 def attention(q, cache_k, cache_v, ctx, group, n_q, n_kv, head_dim, window, scale, chunk=0, keep_first=0,
-              sink_one=False, sink=None, dist_bias=None):
+              sink_one=False, sink=None, dist_bias=None, softcap=0.0):
     """Causal attention of every row over its request's cached keys: all of them, the last `window`, or
     (with `chunk`) those of the row's own chunk of `chunk` positions, chunks counted from position 0.  The
     kernels take the mask as one number: a window as it is, a chunk as its negative.  `keep_first`: beside a
     window, the first that many positions of the sequence stay visible; `sink_one`: the softmax's denominator
     holds one more (a key with score 0 and no value); `sink` [n_q] 32-bit: it holds exp(sink[h]) more instead (a
     learned score of that key, unscaled); `dist_bias` [n_q, L] 32-bit: a number per head and distance query - key
-    added to the scaled score, distances from L - 1 on sharing the last entry."""
+    added to the scaled score, distances from L - 1 on sharing the last entry; `softcap` c > 0: the scaled score s
+    becomes c * tanh(s / c), before the bias."""
     if sink is not None:
         sink_one = False
     if chunk:
@@ -825,10 +829,11 @@ def attention(q, cache_k, cache_v, ctx, group, n_q, n_kv, head_dim, window, scal
         # the denominator's extra one is a sink of 0 for every head
         return attention_tc(q, cache_k, cache_v, ctx.q_start, ctx.kv_len, ctx.pos0, group.block_table,
                             ctx.n_requests, ctx.q_lens, ctx.max_kv_len, n_q, n_kv, head_dim, window, scale,
-                            keep_first=keep_first, dist_bias=dist_bias,
+                            keep_first=keep_first, dist_bias=dist_bias, softcap=softcap,
                             sink=sink if sink is not None else (_zero_sinks(q.device, n_q) if sink_one else None))
     return attention_plain(q, cache_k, cache_v, ctx.row_req, ctx.row_pos, group.block_table, n_q, n_kv, head_dim,
-                           window, scale, keep_first=keep_first, sink_one=sink_one, sink=sink, dist_bias=dist_bias)
+                           window, scale, keep_first=keep_first, sink_one=sink_one, sink=sink, dist_bias=dist_bias,
+                           softcap=softcap)
 
 
 _zero_sink_cache: dict = {}
@@ -1158,7 +1163,8 @@ def latent_attention_plain_form(q: torch.Tensor, cache: torch.Tensor, w_up: torc
     _check(LA.lab_attention_prefill(_ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(pools[0]), _ptr(pools[1]),
                                     _ptr(ctx.q_start), _ptr(ctx.kv_len), _ptr(ctx.pos0), _ptr(table), table.shape[1],
                                     ctx.n_requests, ctx.max_q_len, heads, heads, page_size, num_pages, window,
-                                    ctypes.c_float(scale), int(at_least), _ptr(sink), 0, None, 0, _stream()), "attention_prefill")
+                                    ctypes.c_float(scale), int(at_least), _ptr(sink), 0, None, 0,
+                                    ctypes.c_float(0.0), _stream()), "attention_prefill")
     return out
 
 
@@ -1202,6 +1208,36 @@ def stream_norm_add(x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, eps:
                                                dtype_code(weight.dtype), _stream()),
            "stream_norm_add")
     return rounded
+
+
+def stream_post_norm(x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, alpha: float, eps: float,
+                     copy: bool = False) -> torch.Tensor | None:
+    """x <- rmsnorm(alpha * x + a) * weight in place on the 32-bit stream; `a` is a 32-bit product [tokens, hidden] or
+    split-K partial products [splits, tokens, hidden] (summed in ascending order).  With `copy`, returns the new rows
+    rounded to the weight's storage type."""
+    _on_gpu(x, a, weight)
+    tokens, hidden = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and a.dtype == torch.float32 and a.is_contiguous()
+    assert a.shape[-2:] == x.shape and weight.numel() == hidden
+    rounded = torch.empty((tokens, hidden), dtype=weight.dtype, device=x.device) if copy else None
+    _check(lib("stream32").lab_stream_post_norm(_ptr(x), _ptr(rounded), _ptr(a), a.shape[0] if a.dim() == 3 else 1,
+                                                _ptr(weight), tokens, hidden, ctypes.c_float(alpha), ctypes.c_float(eps),
+                                                dtype_code(weight.dtype), _stream()), "stream_post_norm")
+    return rounded
+
+
+def token_gate(p: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, at: int) -> torch.Tensor:
+    """gelu(p) * table[id, at: at + n] (the tanh form), rounded to the table's storage type: `p` a 32-bit product
+    [tokens, n] or split-K partial products."""
+    _on_gpu(p, table, ids)
+    tokens, n = p.shape[-2:]
+    assert p.dtype == torch.float32 and p.is_contiguous() and table.is_contiguous() and ids.dtype == torch.int32
+    assert ids.numel() >= tokens and 0 <= at and at + n <= table.shape[1]
+    out = torch.empty((tokens, n), dtype=table.dtype, device=p.device)
+    _check(lib("stream32").lab_token_gate(_ptr(out), _ptr(p), p.shape[0] if p.dim() == 3 else 1, _ptr(table), _ptr(ids),
+                                          ctypes.c_longlong(tokens), n, table.shape[1], at, table.shape[0],
+                                          dtype_code(table.dtype), _stream()), "token_gate")
+    return out
 
 
 def stream_round(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
@@ -1299,6 +1335,22 @@ def head_gate(attn: torch.Tensor, proj: torch.Tensor, gate_at: int, per_head: bo
     return out
 
 
+def map_difference(attn: torch.Tensor, heads: int, vdim: int, head: int, lam: float, eps: float, mult: float,
+                   group: int = 0) -> torch.Tensor:
+    """Two score maps' outputs combined per head: a1 - lam * a2 over its root mean square within the head's `vdim`
+    entries (eps inside the root), times `mult`, packed [tokens, heads * vdim] in the storage type of `attn`
+    [tokens, 2 * heads * head].  A head's maps are heads 2h and 2h + 1 of `attn`; `group` > 0 (heads of a group): the
+    queries are ordered by group, map and head within the group."""
+    _on_gpu(attn)
+    tokens = attn.shape[0]
+    assert attn.stride(1) == 1 and attn.shape[1] == 2 * heads * head and vdim <= head
+    out = torch.empty((tokens, heads * vdim), dtype=attn.dtype, device=attn.device)
+    _check(lib("norm_attention").lab_map_difference(
+        _ptr(out), _ptr(attn), attn.stride(0), tokens, heads, vdim, head, int(group > 0), max(int(group), 1),
+        ctypes.c_float(lam), ctypes.c_float(eps), ctypes.c_float(mult), dtype_code(attn.dtype), _stream()), "map_difference")
+    return out
+
+
 # ----------------------------------------------------------------------------------------
 # Recurrent mixers with a scalar decay (csrc/kernels/linear_state.cu).
 # ----------------------------------------------------------------------------------------
@@ -1308,13 +1360,18 @@ def decay_scan_supported(keys: int) -> bool:
 
 def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, ctx, heads: int, groups: int,
                keys: int, vdim: int, a_head: torch.Tensor | None = None, a_tok: torch.Tensor | None = None,
-               s_tok: torch.Tensor | None = None, silu: bool = False, write: bool = True) -> torch.Tensor:
+               s_tok: torch.Tensor | None = None, silu: bool = False, write: bool = True,
+               c_tok: torch.Tensor | None = None) -> torch.Tensor:
     """Per request and head, over the step's rows in order: S <- a S + (s k) v^T, o = S^T q, with S
     [keys, vdim] read from and (with `write`) left in `state` [slots, heads, keys, vdim].  q and k are 32-bit
     column slices [tokens, groups * keys] of one tensor (same row stride), v [tokens, heads * vdim]; `a_head`
     [heads] a fixed decay per head, or `a_tok`/`s_tok` [tokens, heads] per token; `silu`: q, k and v pass a
-    SiLU first.  Returns o [tokens, heads * vdim] in 32-bit."""
-    _on_gpu(q, k, v, state, a_head, a_tok, s_tok)
+    SiLU first.  `c_tok` [tokens, heads], the products q . k, asks for the delta rule: S <- a S, then
+    S <- S + k u^T with u = s (v - S^T k) (`a_tok` and `s_tok` are wanted then).  Returns o [tokens, heads * vdim] in
+    32-bit."""
+    _on_gpu(q, k, v, state, a_head, a_tok, s_tok, c_tok)
+    assert c_tok is None or (a_tok is not None and s_tok is not None and not silu and c_tok.dtype == torch.float32
+                             and c_tok.shape == a_tok.shape and c_tok.stride() == a_tok.stride())
     tokens = v.shape[0]
     for t in (q, k, v):
         assert t.dtype == torch.float32 and t.stride(1) == 1 and t.shape[0] == tokens
@@ -1342,8 +1399,8 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
         vs = 32 if pairs * -(-vdim // 32) >= sm_count() else (16 if pairs * -(-vdim // 16) >= sm_count() else 8)
     vs = min(vs, max(8, 1 << (vdim - 1).bit_length()))
     _check(lib("linear_state").lab_decay_scan(
-        _ptr(out), out.stride(0), _ptr(q), _ptr(k), q.stride(0), _ptr(v), v.stride(0), _ptr(a_tok), _ptr(s_tok), ld_a,
-        _ptr(a_head), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.n_requests, state.shape[0], heads, groups,
+        _ptr(out), out.stride(0), _ptr(q), _ptr(k), q.stride(0), _ptr(v), v.stride(0), _ptr(a_tok), _ptr(s_tok),
+        _ptr(c_tok), ld_a, _ptr(a_head), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.n_requests, state.shape[0], heads, groups,
         keys, vdim, int(silu), int(write), vs, _stream()), "decay_scan")
     return out
 
@@ -1372,6 +1429,54 @@ def ssm_prepare(proj: torch.Tensor, conv_at: int, dt_at: int, channels: int, tap
         tokens, ctx.n_requests, kept.shape[0], int(write), dtype_code(taps_w.dtype), _stream()), "ssm_prepare",
         2 if write and taps > 1 else 1)
     return conv, dt, decay
+
+
+def delta_prepare(proj: torch.Tensor, b_at: int, a_at: int, taps: int, heads: int, groups: int, keys: int, vdim: int,
+                  taps_w: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, kept: torch.Tensor, ctx,
+                  q_scale: float, unit_eps: float, write: bool = True):
+    """What the gated delta rule's recurrence reads, from the 32-bit input projection `proj`: columns [q: groups * keys
+    | k: groups * keys | v: heads * vdim] pass the causal convolution per channel (`taps_w` [channels, taps], no bias;
+    inputs before a request's first row of the step from `kept` [slots, taps - 1, channels], as `ssm_prepare`) and
+    SiLU; q and k become unit vectors per head (`unit_eps` inside the root), q times `q_scale`; columns b_at and a_at
+    on give the rates sigmoid(b) and decays exp(-exp(a_log) softplus(a + dt_bias)).  Returns 32-bit (q, k, v, decay,
+    rate, q . k per head)."""
+    _on_gpu(proj, taps_w, a_log, dt_bias, kept)
+    tokens, gd, hv = proj.shape[0], groups * keys, heads * vdim
+    channels = 2 * gd + hv
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and heads % groups == 0
+    assert proj.shape[1] >= max(channels, b_at + heads, a_at + heads)
+    assert taps_w.shape == (channels, taps) and taps_w.is_contiguous() and a_log.numel() == heads
+    assert dt_bias.numel() == heads and a_log.dtype == taps_w.dtype and dt_bias.dtype == taps_w.dtype
+    assert kept.dtype == torch.float32 and kept.is_contiguous() and tuple(kept.shape[1:]) == (max(taps - 1, 0), channels)
+    if not decay_scan_supported(keys):
+        raise KernelError(f"delta_prepare: {keys} key channels are outside what the recurrence kernel takes (1..256)")
+
+    def new(width):
+        return torch.empty((tokens, width), dtype=torch.float32, device=proj.device)
+
+    q, k, v, decay, rate, qk = new(gd), new(gd), new(hv), new(heads), new(heads), new(heads)
+    _check(lib("linear_state").lab_delta_prepare(
+        _ptr(q), _ptr(k), _ptr(v), _ptr(decay), _ptr(rate), _ptr(qk), _ptr(proj), proj.stride(0), b_at, a_at, taps, heads,
+        groups, keys, vdim, _ptr(taps_w), _ptr(a_log), _ptr(dt_bias), _ptr(kept), _ptr(ctx.row_req), _ptr(ctx.q_start),
+        _ptr(ctx.state_slot), tokens, ctx.n_requests, kept.shape[0], ctypes.c_float(q_scale), ctypes.c_float(unit_eps),
+        int(write), dtype_code(taps_w.dtype), _stream()), "delta_prepare", 2 if write and taps > 1 else 1)
+    return q, k, v, decay, rate, qk
+
+
+def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, ctx, heads: int, vdim: int,
+                   eps: float) -> torch.Tensor:
+    """Every head of `o` [tokens, heads * vdim] (32-bit) over its own root mean square, times `weight` [vdim], times
+    silu(gate) (32-bit column slice of the same shape), rounded to the weight's storage type.  Rows of requests
+    without a state slot (padding) leave as zeros."""
+    _on_gpu(o, gate, weight)
+    tokens = o.shape[0]
+    assert o.dtype == torch.float32 and o.is_contiguous() and o.shape[1] == heads * vdim
+    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == o.shape and weight.numel() == vdim
+    out = torch.empty((tokens, heads * vdim), dtype=weight.dtype, device=o.device)
+    _check(lib("linear_state").lab_head_norm_gate(
+        _ptr(out), _ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(ctx.row_req), _ptr(ctx.state_slot), tokens,
+        heads, vdim, ctypes.c_float(eps), dtype_code(weight.dtype), _stream()), "head_norm_gate")
+    return out
 
 
 def gated_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, parts: int = 1,
@@ -1496,19 +1601,27 @@ MOE_SCORES = {"softmax": 0, "sigmoid": 1}
 
 
 def moe_route(logits: torch.Tensor, experts: int, top: int, gate_col: int = -1, renorm: bool = True,
-              score: str = "softmax"):
+              score: str = "softmax", correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1,
+              scale: float = 1.0):
     """From 32-bit router logits [tokens, >= experts] (column `gate_col` >= 0: the logit of a shared expert's
     gate): (chosen experts [tokens, top] int32, their weights [tokens, top], sigmoid of the gate's logit
     [tokens] or None).  The scores are the softmax over all experts or (`score` "sigmoid") the sigmoid of each
-    logit; the weights are the chosen scores over their sum, or (`renorm` False) as they are."""
-    _on_gpu(logits)
+    logit; the weights are the chosen scores over their sum, or (`renorm` False) as they are, times `scale`.
+    `correction` [experts] 32-bit joins the scores for the choice alone.  `groups` > 1: the experts lie in that many
+    equal groups of neighbours, and only those of the `keep` groups whose largest choice score is largest can be
+    chosen."""
+    _on_gpu(logits, correction)
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
+    if experts % groups or not 1 <= keep <= groups or top > keep * (experts // groups):
+        raise KernelError(f"moe_route: {top} of {experts} experts in {groups} groups of which {keep} are kept")
     tokens = logits.shape[0]
     assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= experts
     chosen = torch.empty((tokens, top), dtype=torch.int32, device=logits.device)
     weight = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     gate = torch.empty((tokens,), dtype=torch.float32, device=logits.device) if gate_col >= 0 else None
     _check(lib("moe").lab_moe_route(_ptr(chosen), _ptr(weight), _ptr(gate), _ptr(logits), logits.stride(0), tokens,
-                                    experts, top, gate_col, int(bool(renorm)), MOE_SCORES[score], _stream()),
+                                    experts, top, gate_col, int(bool(renorm)), MOE_SCORES[score], _ptr(correction),
+                                    int(groups), int(keep), ctypes.c_float(scale), _stream()),
            "moe_route")
     return chosen, weight, gate
 
@@ -1533,18 +1646,44 @@ def moe_align(chosen: torch.Tensor, experts: int, tile: int):
 
 
 def moe_combine(y: torch.Tensor, pos_of: torch.Tensor, weight: torch.Tensor | None, shared: torch.Tensor | None,
-                shared_gate: torch.Tensor | None, top: int | None = None) -> torch.Tensor:
+                shared_gate: torch.Tensor | None, top: int | None = None, chosen: torch.Tensor | None = None,
+                identity_from: int = 0, h: torch.Tensor | None = None) -> torch.Tensor:
     """out[t] = sum_k weight[t, k] * y[pos_of[t, k]] (+ shared_gate[t] * shared[t]), 32-bit.  `weight` None: the plain
-    sum over each token's `top` pairs."""
-    _on_gpu(y, pos_of, weight, shared, shared_gate)
+    sum over each token's `top` pairs.  `chosen` [tokens, top] with `identity_from` and the layer's input `h`: experts
+    from that index on give h back."""
+    _on_gpu(y, pos_of, weight, shared, shared_gate, chosen, h)
+    assert chosen is None or (chosen.dtype == torch.int32 and h.is_contiguous() and h.shape[1] == y.shape[1])
     tokens, top = weight.shape if weight is not None else (pos_of.numel() // top, top)
     width = y.shape[1]
     assert y.dtype == torch.float32 and y.is_contiguous() and (weight is None or weight.dtype == torch.float32)
     assert shared is None or (shared.dtype == torch.float32 and shared.is_contiguous() and shared.shape == (tokens, width))
     out = torch.empty((tokens, width), dtype=torch.float32, device=y.device)
     _check(lib("moe").lab_moe_combine(_ptr(out), _ptr(y), _ptr(pos_of), _ptr(weight), _ptr(shared), _ptr(shared_gate),
-                                      tokens, top, width, _stream()), "moe_combine")
+                                      tokens, top, width, _ptr(chosen), int(identity_from), _ptr(h),
+                                      dtype_code(h.dtype) if h is not None else F32, _stream()), "moe_combine")
     return out
+
+
+def moe_combine_norm(x: torch.Tensor, y: torch.Tensor, pos_of: torch.Tensor, weight: torch.Tensor, chosen: torch.Tensor,
+                     identity_from: int, shared: torch.Tensor | None, shared_gate: torch.Tensor | None,
+                     norm_weight: torch.Tensor, alpha: float, eps: float, copy: bool = False) -> torch.Tensor | None:
+    """x <- rmsnorm(alpha * x + the weighted sum) * norm_weight in place on the 32-bit stream, the sum as `moe_combine`
+    forms it (`shared` may be split-K partial products) with the identity experts' weights on x itself.  With `copy`,
+    returns the new rows rounded to the weight's storage type."""
+    _on_gpu(x, y, pos_of, weight, chosen, shared, shared_gate, norm_weight)
+    (tokens, width), top = x.shape, chosen.shape[1]
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.dtype == torch.float32 and y.is_contiguous()
+    assert y.shape[1] == width and pos_of.numel() == tokens * top and chosen.dtype == torch.int32
+    assert weight is None or (weight.dtype == torch.float32 and weight.shape == chosen.shape)
+    assert shared is None or (shared.dtype == torch.float32 and shared.is_contiguous() and shared.shape[-2:] == x.shape)
+    assert norm_weight.numel() == width
+    rounded = torch.empty((tokens, width), dtype=norm_weight.dtype, device=x.device) if copy else None
+    _check(lib("moe").lab_moe_combine_norm(
+        _ptr(x), _ptr(rounded), _ptr(y), _ptr(pos_of), _ptr(weight), _ptr(chosen), int(identity_from), _ptr(shared),
+        shared.shape[0] if shared is not None and shared.dim() == 3 else 1, _ptr(shared_gate), _ptr(norm_weight), tokens,
+        top, width, ctypes.c_float(alpha), ctypes.c_float(eps), dtype_code(norm_weight.dtype), _stream()),
+        "moe_combine_norm")
+    return rounded
 
 
 GROUPED_KERNEL = "auto"     # "auto", "tc" (tcgen05, rows gathered first), "plain" (ordinary units) or "tiles" (their tiled kernel only)
@@ -1693,12 +1832,17 @@ def linear_grouped(x: torch.Tensor, w: torch.Tensor, row_src: torch.Tensor | Non
 def head_prep_store(proj: torch.Tensor, bias, positions: torch.Tensor, inv_freq: torch.Tensor | None, rot_dims: int, slots,
                     cache_k, cache_v, n_q: int, n_kv: int, dim: int, vdim: int, head: int, k_at: int, v_at: int,
                     dtype: torch.dtype, norm_eps: float = 0.0, q_norm_w=None, k_norm_w=None, q_head_scale=None,
-                    temp_coef: float = 0.0, temp_every: int = 0) -> torch.Tensor:
+                    temp_coef: float = 0.0, temp_every: int = 0, maps: int = 1, v_rep: int = 1) -> torch.Tensor:
     """`rope_pairs_store` with a norm per head and temperatures on q: after the rotation (`rot_dims` 0: none) every q
     and k head is divided by its root mean square over `dim` (`norm_eps` > 0; eps inside the root) and multiplied by
     a weight of `dim` entries shared by the heads (`q_norm_w`, `k_norm_w`; None: no weight); q is then multiplied by
     `q_head_scale` [n_q] (32-bit; None: 1) and, with `temp_every` > 0, by 1 + temp_coef * ln(floor((pos + 1) /
-    temp_every) + 1).  Everything in 32-bit; one rounding where q, k and v leave."""
+    temp_every) + 1).  Everything in 32-bit; one rounding where q, k and v leave.
+
+    `maps` M > 1: every key/value head holds M keys side by side (M * dim <= head; the projection has n_kv * M keys,
+    head by head), n_q counts heads and maps together, and query i lies at the entries of key i % M of its head with
+    zeros elsewhere.  `v_rep` R > 1: the projection has n_kv / R value heads, key head g is stored with value head
+    g // R."""
     _on_gpu(proj, bias, positions, inv_freq, slots, cache_k, cache_v, q_norm_w, k_norm_w, q_head_scale)
     splits = proj.shape[0] if proj.dim() == 3 else 1
     tokens, ld = proj.shape[-2], proj.stride(-2)       # a column slice of a wider product will do
@@ -1721,7 +1865,7 @@ def head_prep_store(proj: torch.Tensor, bias, positions: torch.Tensor, inv_freq:
         ctypes.c_longlong(tokens * ld), ld, k_at, v_at, _ptr(bias), _ptr(positions), _ptr(inv_freq), rot_dims,
         _ptr(slots), ctypes.c_longlong(n_slots), tokens, n_q, n_kv, dim, vdim, head, max(page_size, 1),
         ctypes.c_float(norm_eps), _ptr(q_norm_w), _ptr(k_norm_w), _ptr(q_head_scale), ctypes.c_float(temp_coef),
-        int(temp_every), dtype_code(dtype), _stream()), "head_prep_store")
+        int(temp_every), int(maps), int(v_rep), dtype_code(dtype), _stream()), "head_prep_store")
     return q
 
 

@@ -8,7 +8,7 @@ import torch
 
 from ..kernels import ops
 from ..profiling import scoped_range
-from .base import Block, register_part
+from .base import Block, lookup, register_part
 from .norm import StreamRMSNorm
 from .spec import FixedState, TensorSpec
 
@@ -270,3 +270,77 @@ class SandwichStreamBlock(Block):
 
 
 register_part("block", "sandwich_stream", SandwichStreamBlock)
+
+
+class PostNormBlock(Block):
+    """The 32-bit stream itself is normed after every sum, with `alpha` on what was there before:
+
+        x <- norm1(alpha x + mixer(x));   x <- norm2(alpha x + ffn(x))
+
+    (RMS norms with plain weights; a layer may have no feed-forward: one norm then.)  The sublayers read x itself.
+    With `side`, a feed-forward spec, a third sublayer's output is normed and added last: x <- x + norm3(side(x)),
+    its norm the last of the block's norms.
+
+    The sublayers' products arrive in 32-bit, whole or as split-K partial products; one kernel sums them into the
+    stream, norms it and leaves the new rows rounded for the product that reads them next.  A feed-forward that forms
+    its result from many parts (`forward_post_norm`) does so in that pass.  The block owes the stream nothing
+    (`RoundedStream`)."""
+    decode_graph_safe = True
+
+    n_norms = 3
+
+    @classmethod
+    def tensors(cls, spec):
+        side = spec.get("side") if spec is not None else None
+        return lookup("feed_forward", side.kind).tensors(side) if side is not None else []
+
+    @classmethod
+    def libraries(cls, spec, dtype):
+        side = spec.get("side") if spec is not None else None
+        return [("stream32", {})] + (lookup("feed_forward", side.kind).libraries(side, dtype) if side is not None else [])
+
+    def __init__(self, mixer, ffn, norms, spec=None, weights=None, dtype=None, device=None):
+        super().__init__(mixer, ffn, norms, spec, weights, dtype, device)
+        if spec is None:
+            raise ValueError("postnorm_stream: the block needs a spec (alpha)")
+        self.dtype, self.alpha = dtype, float(spec["alpha"])
+        side = spec.get("side")
+        self.side = lookup("feed_forward", side.kind)(side, weights, dtype, device) if side is not None else None
+        want = 1 + (ffn is not None) + (side is not None)
+        if len(norms) != want or any(type(n) is not StreamRMSNorm or n.offset != 0.0 for n in norms):
+            raise ValueError(f"postnorm_stream: {want} norms, rmsnorm_stream with plain weights")
+        self.side_range = "feed_forward." + (side.kind if side is not None else "none")
+
+    def forward(self, x, pending, ctx, cache):
+        copy = self.dtype != torch.float32
+        if isinstance(pending, RoundedStream):
+            h = pending.rows
+        else:
+            if pending is not None:
+                if not hasattr(pending, "add_to"):
+                    raise ValueError("postnorm_stream follows a block whose sum it cannot take")
+                pending.add_to(x)
+            h = ops.stream_round(x, self.dtype)
+
+        def rows(rounded):      # what the next sublayer reads: in a 32-bit engine the stream itself
+            return x if rounded is None else rounded
+
+        n1 = self.norms[0]
+        with scoped_range(self.mixer_range):
+            a = self.mixer.forward(h, ctx, cache)
+            h = rows(ops.stream_post_norm(x, a, n1.weight, self.alpha, n1.eps, copy=copy))
+        if self.ffn is not None:
+            n2 = self.norms[1]
+            with scoped_range(self.ffn_range):
+                if hasattr(self.ffn, "forward_post_norm"):
+                    h = rows(self.ffn.forward_post_norm(x, h, ctx, n2.weight, self.alpha, n2.eps, copy))
+                else:
+                    h = rows(ops.stream_post_norm(x, self.ffn.forward(h, ctx), n2.weight, self.alpha, n2.eps, copy=copy))
+        if self.side is not None:
+            n3 = self.norms[-1]
+            with scoped_range(self.side_range):
+                h = rows(ops.stream_norm_add(x, self.side.forward(h, ctx), n3.weight, n3.eps, copy=copy))
+        return x, RoundedStream(h)
+
+
+register_part("block", "postnorm_stream", PostNormBlock)

@@ -1,4 +1,5 @@
-"""Recurrent mixer: the generalized delta rule."""
+"""Recurrent mixers by the delta rule: the generalized rule with decays per channel, and the gated rule with one decay
+per head."""
 from __future__ import annotations
 
 import math
@@ -7,7 +8,7 @@ import torch
 
 from ..kernels import ops
 from .base import CacheView, Mixer, StepContext, register_part
-from .spec import FixedState, PartSpec, TensorSpec
+from .spec import CacheParts, FixedState, PartSpec, TensorSpec
 
 
 class GeneralDelta(Mixer):
@@ -71,3 +72,84 @@ class GeneralDelta(Mixer):
 
 
 register_part("mixer", "general_delta", GeneralDelta)
+
+
+class GatedDelta(Mixer):
+    """The gated delta rule with short convolutions.  q = W_q h, k = W_k h (`kv_heads` x `dim`), v = W_v h (`heads` x
+    `vdim`); head h reads the q and k of group h // (heads / kv_heads).  Every channel of q, k and v passes a causal
+    convolution over its last `taps` inputs (tensors `q.conv`, `k.conv`, `v.conv` [channels, taps], the last column on
+    the current token, no bias, zeros before the sequence) and SiLU.  q and k become unit vectors per head, x /
+    sqrt(sum x^2 + `unit_eps`), q times dim^(-1/2).  Per head, with the rate beta = sigmoid(W_b h) and the decay
+    g = exp(-exp(A_log) softplus(W_a h + dt_bias)):
+
+        S <- g S;   S <- S + k (beta (v - S^T k))^T;   o = S^T q
+
+    Each head's o over its root mean square (`eps`), times a weight of `vdim` entries all heads share, times
+    silu(W_g h); W_o closes.  Per request the mixer keeps S (32-bit) and the convolutions' last taps - 1 inputs: two
+    fixed-size states (`CacheParts`).
+
+    The matrices that read h are one product, taken in 32-bit; one kernel convolves, forms the unit vectors, rates
+    and decays, one walks the state (`ops.decay_scan`), one norms and gates.  All of it is 32-bit up to the rounding
+    before W_o."""
+    decode_graph_safe = True
+    CONVOLVED = ("q", "k", "v")
+
+    @classmethod
+    def _sizes(cls, spec):
+        return spec["kv_heads"] * spec["dim"], spec["heads"] * spec["vdim"]
+
+    @classmethod
+    def tensors(cls, spec: PartSpec):
+        h, H, p = spec["hidden"], spec["heads"], spec.prefix
+        gd, hv = cls._sizes(spec)
+        out = []
+        for n, rows in zip(cls.CONVOLVED, (gd, gd, hv)):
+            out += [TensorSpec(p + n, (rows, h)), TensorSpec(p + n + ".conv", (rows, spec["taps"]))]
+        out += [TensorSpec(p + "g", (hv, h)), TensorSpec(p + "b", (H, h)), TensorSpec(p + "a", (H, h)),
+                TensorSpec(p + "A_log", (H,), init="bias"), TensorSpec(p + "dt_bias", (H,), init="bias"),
+                TensorSpec(p + "norm", (spec["vdim"],), init="norm"), TensorSpec(p + "o", (h, hv))]
+        return out
+
+    @classmethod
+    def cache_need(cls, spec: PartSpec):
+        gd, hv = cls._sizes(spec)
+        return CacheParts((FixedState((spec["heads"], spec["dim"], spec["vdim"])),
+                           FixedState((max(spec["taps"] - 1, 0), 2 * gd + hv))))
+
+    @classmethod
+    def libraries(cls, spec, dtype):
+        return [("linear_state", {})]
+
+    def __init__(self, spec, weights, dtype, device):
+        super().__init__(spec, weights, dtype, device)
+        self.heads, self.groups, self.dim, self.vdim, self.taps = (
+            int(spec[k]) for k in ("heads", "kv_heads", "dim", "vdim", "taps"))
+        if self.heads % self.groups:
+            raise ValueError("gated_delta: heads must be a multiple of kv_heads")
+        if not ops.decay_scan_supported(self.dim):
+            raise ValueError(f"gated_delta: {self.dim} key channels are outside what the recurrence kernel takes")
+        self.eps, self.unit_eps = float(spec["eps"]), float(spec.get("unit_eps", 1e-6))
+        w = lambda n: self._weight(weights, n)  # noqa: E731
+        self.gd, self.hv = self._sizes(spec)
+        self.w_in = torch.cat([w(n) for n in ("q", "k", "v", "g", "b", "a")], dim=0).contiguous()
+        self.gate_at = 2 * self.gd + self.hv
+        self.rate_at = self.gate_at + self.hv
+        self.decay_at = self.rate_at + self.heads
+        self.conv_w = torch.cat([w(n + ".conv") for n in self.CONVOLVED], dim=0).contiguous()
+        self.a_log, self.dt_bias, self.norm_weight = w("A_log"), w("dt_bias"), w("norm")
+        self.w_o = w("o").contiguous()
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+        proj = ops.linear(x, self.w_in, None, out_f32=True)
+        state, kept = cache.part(0), cache.part(1)
+        q, k, v, decay, rate, qk = ops.delta_prepare(
+            proj, self.rate_at, self.decay_at, self.taps, self.heads, self.groups, self.dim, self.vdim, self.conv_w,
+            self.a_log, self.dt_bias, kept.state, ctx, self.dim ** -0.5, self.unit_eps, write=cache.write)
+        o = ops.decay_scan(q, k, v, state.state, ctx, self.heads, self.groups, self.dim, self.vdim, a_tok=decay,
+                           s_tok=rate, c_tok=qk, write=cache.write)
+        y = ops.head_norm_gate(o, proj[:, self.gate_at: self.gate_at + self.hv], self.norm_weight, ctx, self.heads,
+                               self.vdim, self.eps)
+        return ops.linear(y, self.w_o, None, out_f32=True, allow_partial=True)
+
+
+register_part("mixer", "gated_delta", GatedDelta)

@@ -45,8 +45,8 @@ class NormedTokenEmbedding(Embedding):
 
 
 class TokenPositionEmbedding(Embedding):
-    """x[t] = table[id_t] + positions[p_t] as a 32-bit residual stream: a learned vector per absolute
-    position (the table's rows bound the longest sequence), added unscaled."""
+    """x[t] = table[id_t] * `scale` (1 where none is given) + positions[p_t] as a 32-bit residual stream: a learned
+    vector per absolute position (the table's rows bound the longest sequence), added unscaled."""
 
     @classmethod
     def tensors(cls, spec: PartSpec):
@@ -64,11 +64,12 @@ class TokenPositionEmbedding(Embedding):
         weights[spec["table"]] = self.table      # a tied head shares this storage
         p = weights[spec["positions"]]
         self.positions = (p if p.dtype == dtype else p.to(dtype)).contiguous()
+        self.scale = float(spec.get("scale", 1.0))
 
     def forward(self, token_ids, positions=None):
         if positions is None:
             raise ValueError("token_position_embedding needs the rows' positions")
-        return ops.embed_position(token_ids, positions, self.table, self.positions)
+        return ops.embed_position(token_ids, positions, self.table, self.positions, scale=self.scale)
 
 
 class StreamTokenEmbedding(Embedding):

@@ -19,14 +19,20 @@ class RoutedExperts(FeedForward):
     capped form W_down (g' * sigmoid(1.702 g') * (u' + 1)) with g' = min(W_gate h, limit) and u' = clamp(W_up h,
     -limit, limit).
 
+    `correction` True: a learned number per expert (tensor `correction`) joins the scores for the choice, not for the
+    weights.  `groups` (count, keep): the experts form `count` equal groups of neighbours and only those of the `keep`
+    groups whose largest choice score is largest can be chosen.  `identity` > 0: the router has that many more
+    outputs, identity experts without matrices whose result is h itself.  `router_scale` multiplies the weights.
+
     The router's matrix and the gate's row are one product; one kernel picks, one lays the (token, expert)
     pairs out in rows grouped by expert, two grouped products run the experts, and one kernel forms the weighted
     sum, in the order of each token's choice, with the shared expert's share.  Steps of many pairs in bfloat16
     run the grouped products on the tensor cores over rows gathered into the layout; else the ordinary units
-    gather while they load.  The result is 32-bit."""
+    gather while they load.  The result is 32-bit.  `forward_post_norm` leaves the weighted sum in a 32-bit stream
+    that is normed as a whole, in one pass."""
 
     NAMES = {"router": "router", "expert": "e{}.", "gate": "gate", "up": "up", "down": "down", "shared": "shared.",
-             "shared_gate": "shared.sg"}
+             "shared_gate": "shared.sg", "correction": "correction"}
 
     @classmethod
     def names(cls, spec: PartSpec) -> dict:
@@ -35,7 +41,10 @@ class RoutedExperts(FeedForward):
     @classmethod
     def tensors(cls, spec: PartSpec):
         h, E, F, p, n = spec["hidden"], spec["experts"], spec["expert_ff"], spec.prefix, cls.names(spec)
-        out = [TensorSpec(p + n["router"], (E, h))]
+        outputs = E + int(spec.get("identity") or 0)
+        out = [TensorSpec(p + n["router"], (outputs, h))]
+        if spec.get("correction"):
+            out.append(TensorSpec(p + n["correction"], (outputs,), init="bias"))
         for e in range(E):
             q = p + n["expert"].format(e)
             out += [TensorSpec(q + n["gate"], (F, h)), TensorSpec(q + n["up"], (F, h)), TensorSpec(q + n["down"], (h, F))]
@@ -54,8 +63,15 @@ class RoutedExperts(FeedForward):
     def __init__(self, spec, weights, dtype, device):
         super().__init__(spec, weights, dtype, device)
         self.experts, self.top, self.ff = int(spec["experts"]), int(spec["top"]), int(spec["expert_ff"])
-        if not 0 < self.top <= self.experts:
+        self.identity = int(spec.get("identity") or 0)
+        self.outputs = self.experts + self.identity
+        self.groups, self.keep = (int(g) for g in (spec.get("groups") or (1, 1)))
+        self.router_scale = float(spec.get("router_scale", 1.0))
+        if not 0 < self.top <= self.outputs:
             raise ValueError("routed_experts: top must lie in 1..experts")
+        if self.outputs % self.groups or not 1 <= self.keep <= self.groups or \
+                self.top > self.keep * (self.outputs // self.groups):
+            raise ValueError("routed_experts: groups must divide the experts, and the kept ones hold at least top experts")
         n = self.names(spec)
         w = lambda name: self._weight(weights, name)  # noqa: E731
         self.shared_ff = int(spec.get("shared_ff") or 0)
@@ -68,6 +84,11 @@ class RoutedExperts(FeedForward):
         self.limit, self.shared_limit = float(spec.get("limit") or 0.0), float(spec.get("shared_limit") or 0.0)
         rows = [w(n["router"])] + ([w(n["shared_gate"]).reshape(1, -1)] if self.gated_share else [])
         self.w_router = torch.cat(rows, dim=0).contiguous()
+        self.correction = None
+        if spec.get("correction"):
+            self.correction = weights[spec.prefix + n["correction"]].to(device=device, dtype=torch.float32).contiguous()
+        if self.scale_input and self.identity:
+            raise ValueError("routed_experts: identity experts go with weights on the experts' outputs")
         names = [n["expert"].format(e) for e in range(self.experts)]
         self.w_gate_up = torch.stack([torch.cat([w(q + n["gate"]), w(q + n["up"])], dim=0) for q in names]).contiguous()
         self.w_down = torch.stack([w(q + n["down"]) for q in names]).contiguous()
@@ -76,20 +97,35 @@ class RoutedExperts(FeedForward):
             self.w_shared_gate_up = torch.cat([w(q + n["gate"]), w(q + n["up"])], dim=0).contiguous()
             self.w_shared_down = w(q + n["down"]).contiguous()
 
-    def forward(self, x, ctx):
+    def _experts(self, x):
+        """The choice and the chosen experts' results: (chosen, weights, shared gate, layout, results by layout row)."""
         E, top = self.experts, self.top
         logits = ops.linear(x, self.w_router, None, out_f32=True)
-        chosen, weight, gate = ops.moe_route(logits, E, top, gate_col=E if self.gated_share else -1, renorm=self.renorm,
-                                             score=self.score)
+        chosen, weight, gate = ops.moe_route(logits, self.outputs, top, gate_col=self.outputs if self.gated_share else -1,
+                                             renorm=self.renorm, score=self.score, correction=self.correction,
+                                             groups=self.groups, keep=self.keep, scale=self.router_scale)
         lay = ops.moe_layout(chosen, E, x.dtype, x.shape[1], self.ff)
         act = ops.moe_experts_up(x, self.w_gate_up, lay, top, limit=self.limit,
                                  in_scale=weight if self.scale_input else None)
-        y = ops.moe_experts_down(act, self.w_down, lay)
-        shared = None
-        if self.shared_ff:
-            shared = ops.linear(ops.linear_gated(x, self.w_shared_gate_up, limit=self.shared_limit), self.w_shared_down,
-                                None, out_f32=True)
-        return ops.moe_combine(y, lay.pos_of, None if self.scale_input else weight, shared, gate, top=top)
+        return chosen, None if self.scale_input else weight, gate, lay, ops.moe_experts_down(act, self.w_down, lay)
+
+    def _shared(self, x, allow_partial=False):
+        if not self.shared_ff:
+            return None
+        return ops.linear(ops.linear_gated(x, self.w_shared_gate_up, limit=self.shared_limit), self.w_shared_down,
+                          None, out_f32=True, allow_partial=allow_partial)
+
+    def forward(self, x, ctx):
+        chosen, weight, gate, lay, y = self._experts(x)
+        more = {"chosen": chosen, "identity_from": self.experts, "h": x} if self.identity else {}
+        return ops.moe_combine(y, lay.pos_of, weight, self._shared(x), gate, top=self.top, **more)
+
+    def forward_post_norm(self, stream, x, ctx, weight, alpha, eps, copy):
+        """stream <- rmsnorm(alpha * stream + the layer's result on x) * weight, x the stream's rows rounded; identity
+        experts give the stream's own 32-bit rows.  Returns the new rows rounded with `copy`."""
+        chosen, w, gate, lay, y = self._experts(x)
+        return ops.moe_combine_norm(stream, y, lay.pos_of, w, chosen, self.experts, self._shared(x, allow_partial=True),
+                                    gate, weight, alpha, eps, copy=copy)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

@@ -76,6 +76,8 @@ def _register_builtin() -> None:
     register_architecture("Kupedra", KupedraConfig, kupedra_blueprint)
     from .config.difedra import DifedraConfig, difedra_blueprint
     register_architecture("Difedra", DifedraConfig, difedra_blueprint)
+    from .config.nudusun import NudusunConfig, nudusun_blueprint
+    register_architecture("Nudusun", NudusunConfig, nudusun_blueprint)
 
 
 _register_builtin()
