@@ -1296,6 +1296,201 @@ def run_arch_difedra(args):
     return 0
 
 
+# ----------------------------------------------------------------------------------------
+# --arch nudusun: the Nudusun design beside Kupedra and Qwen2 at equal layer sizes (random weights)
+# ----------------------------------------------------------------------------------------
+NUDUSUN_SHAPES = {
+    # width and vocabulary of the Qwen2.5 shape of the same name; differential attention with heads x vdim = width and
+    # as many score maps as Qwen2 has heads of 64; the delta rule with heads x vdim = width; experts as in the Kupedra
+    # shape of the same name, with four identity experts beside them
+    "0.5B": dict(heads=7, kv_heads=1, dim=64, vdim=128, window=1024, del_heads=14, del_kv=7, del_dim=64, del_vdim=64,
+                 taps=4, experts=8, identity=4, top=3, groups=4, keep=3, expert_ff=1536, shared_ff=1792, side=64),
+    "1.5B": dict(heads=12, kv_heads=2, dim=64, vdim=128, window=2048, del_heads=12, del_kv=6, del_dim=128, del_vdim=128,
+                 taps=4, experts=8, identity=4, top=3, groups=4, keep=3, expert_ff=2816, shared_ff=3328, side=96),
+}
+
+
+def nudusun_config(shape, layers):
+    """Layers alternate: the gated delta rule, then differential attention; every layer with routed experts."""
+    q, m = SHAPES[shape], NUDUSUN_SHAPES[shape]
+    moe = {"kind": "moe", "expert": {"ff": m["expert_ff"], "limit": 7.0}, "shared": {"ff": m["shared_ff"], "limit": 7.0},
+           "router": {"experts": m["experts"], "identity": m["identity"], "top": m["top"], "scale": 1.5,
+                      "groups": {"count": m["groups"], "keep": m["keep"]}}}
+    kinds = [{"type": "delta", "mlp": moe,
+              "mixer": {"heads": m["del_heads"], "kv_heads": m["del_kv"], "dim": m["del_dim"], "vdim": m["del_vdim"],
+                        "conv": m["taps"]}},
+             {"type": "attention", "mlp": moe,
+              "mixer": {"heads": m["heads"], "kv_heads": m["kv_heads"], "dim": m["dim"], "vdim": m["vdim"],
+                        "scale": m["dim"] ** -0.5, "softcap": 50.0, "diff": 0.4, "mask": {"size": m["window"]}}}]
+    return {"architecture": "Nudusun", "vocab": q["vocab_size"], "width": q["hidden_size"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "postln_alpha": 2.0, "token_side": {"dim": m["side"]}, "max_positions": 4096,
+            "layers": [kinds[i % 2] for i in range(layers)]}
+
+
+def kernel_points_nudusun(shape, batch, ctx_len, prefill_tokens, pk):
+    """The Nudusun design's own kernels beside the like kernels of Sogulix (the delta rule), of Ritizen (the recurrence
+    and its preparation, the gate on the heads), of Kupedra (the attention's store, the router, the matrix memory) and
+    of Bukatar (the sums that close a sublayer) at the shape's sizes, each alone between CUDA events with L2 flushed:
+    milliseconds and the fraction of the roofline (measured copy bandwidth for kernels that stream, measured bf16
+    product rate for the attention kernels and the products of a prompt)."""
+    import torch
+    from llm_inference_lab_b200.kernels import ops
+
+    dev = torch.device("cuda:0")
+    q, m = SHAPES[shape], NUDUSUN_SHAPES[shape]
+    width = q["hidden_size"]
+    flush = torch.zeros((160 << 20,), dtype=torch.int16, device=dev)
+    bw, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    rows = {}
+
+    def record(name, ms, nbytes=None, flops=None):
+        entry = {"ms": round(ms, 4)}
+        if nbytes is not None:
+            entry.update(gbs=round(nbytes / (ms / 1e3) / 1e9, 1), frac_hbm=round(nbytes / (ms / 1e3) / bw, 4))
+        if flops is not None:
+            entry.update(tflops=round(flops / (ms / 1e3) / 1e12, 2), frac_bf16=round(flops / (ms / 1e3) / tf, 4))
+        rows[name] = entry
+
+    bf = lambda *s: (0.5 * torch.randn(*s, device=dev)).to(torch.bfloat16)  # noqa: E731
+    f32 = lambda *s: 0.5 * torch.randn(*s, device=dev)  # noqa: E731
+    for label, q_lens, pos0 in (("prefill", [prefill_tokens], [0]), ("decode", [1] * batch, [ctx_len] * batch)):
+        T, B = sum(q_lens), len(q_lens)
+        ctx, pages = bench_ctx(q_lens, pos0, PAGE_SIZE, dev)
+        slots = ctx.groups[0].row_slot
+        prompt = label == "prefill"
+        # ---- the gated delta rule: preparation, walk, norm and gate; beside the generalized delta rule (Sogulix; its
+        # heads are square, so at the same key size) and the walk without the rule (Ritizen, Kupedra)
+        H, G, D, V, K = m["del_heads"], m["del_kv"], m["del_dim"], m["del_vdim"], m["taps"]
+        gd, hv = G * D, H * V
+        ch = 2 * gd + hv
+        proj = f32(T, ch + hv + 2 * H)
+        conv_w, hb, w_v = bf(ch, K), bf(H), bf(V)
+        state, kept = torch.zeros(B, H, D, V, device=dev), torch.zeros(B, K - 1, ch, device=dev)
+
+        def prepare():
+            return ops.delta_prepare(proj, ch + hv, ch + hv + H, K, H, G, D, V, conv_w, hb, hb, kept, ctx, D ** -0.5, 1e-6)
+
+        dq, dk, dv, decay, rate, qk = prepare()
+        walk = lambda: ops.decay_scan(dq, dk, dv, state, ctx, H, G, D, V, a_tok=decay, s_tok=rate, c_tok=qk)  # noqa: E731
+        o = walk()
+        gate = proj[:, ch: ch + hv]
+        finish = lambda: ops.head_norm_gate(o, gate, w_v, ctx, H, V, 1e-6)  # noqa: E731
+        prep_bytes = T * (2 * ch + 5 * H) * 4 + B * (K - 1) * ch * 8
+        walk_bytes = T * (2 * gd + 2 * hv + 3 * H) * 4 + 2 * state.numel() * 4
+        walk_flops = 6.0 * T * H * D * V if prompt else None
+        record(f"delta_prepare {label}", timed(prepare, flush=flush), nbytes=prep_bytes)
+        record(f"gated delta rule, the walk {label}", timed(walk, flush=flush), nbytes=walk_bytes, flops=walk_flops)
+        record(f"head_norm_gate {label}", timed(finish, flush=flush), nbytes=T * hv * (4 + 4 + 2))
+
+        def whole():
+            a = prepare()
+            ops.decay_scan(a[0], a[1], a[2], state, ctx, H, G, D, V, a_tok=a[3], s_tok=a[4], c_tok=a[5])
+            finish()
+
+        record(f"gated delta rule, all of it {label}", timed(whole, flush=flush),
+               nbytes=prep_bytes + walk_bytes + T * hv * 10, flops=walk_flops)
+        sproj, dpre, ones = f32(T, 5 * H * D), f32(T, H * D), bf(H * D)
+        square = torch.zeros(B, H, D, D, device=dev)
+        ms = timed(lambda: ops.delta_rule(sproj, dpre, ones, ones, ones, square, ctx, H, D, 1e-6, 0.6), flush=flush)
+        record(f"sogulix delta_rule, all of it {label}", ms, nbytes=T * H * D * (6 * 4 + 2) + 2 * square.numel() * 4,
+               flops=8.0 * T * H * D * D if prompt else None)
+        ms = timed(lambda: ops.decay_scan(dq, dk, dv, state, ctx, H, G, D, V, a_tok=decay, s_tok=rate), flush=flush)
+        record(f"ritizen decay_scan decay per token {label}", ms, nbytes=walk_bytes,
+               flops=4.0 * T * H * D * V if prompt else None)
+        ms = timed(lambda: ops.ssm_prepare(proj, 0, ch + hv, ch, K, H, conv_w, conv_w[:, 0].contiguous(), hb, hb, kept, ctx),
+                   flush=flush)
+        record(f"ritizen ssm_prepare {label}", ms, nbytes=prep_bytes)
+        w_hv = bf(hv)
+        ms = timed(lambda: ops.gated_norm(o, gate, w_hv, 1e-6), flush=flush)
+        record(f"ritizen gated_norm {label}", ms, nbytes=T * hv * (4 + 4 + 2))
+        # ---- differential attention: the store of two maps a head beside one norm per head (Kupedra), the kernels with
+        # and without a cap on the scores, the maps' difference beside the gate on the heads (Ritizen)
+        nq, nkv, D, V, win = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["window"]
+        hd = ops.padded_head(2 * D, V)
+        ck, cv, wn = bf(pages, nkv, PAGE_SIZE, hd), bf(pages, nkv, PAGE_SIZE, hd), bf(D)
+        aproj = f32(T, 2 * (nq + nkv) * D + nkv * V)
+        io = T * ((2 * (nq + nkv) * D + nkv * V) * 4 + (2 * nq + 2 * nkv) * hd * 2)
+        ms = timed(lambda: ops.head_prep_store(aproj, None, ctx.row_pos, None, 0, slots, ck, cv, 2 * nq, nkv, D, V, hd,
+                                               2 * nq * D, 2 * (nq + nkv) * D, torch.bfloat16, norm_eps=1e-6, q_norm_w=wn,
+                                               k_norm_w=wn, maps=2), flush=flush)
+        record(f"head_prep_store two maps {label}", ms, nbytes=io)
+        ck1, cv1, wn1 = bf(pages, 2 * nkv, PAGE_SIZE, D), bf(pages, 2 * nkv, PAGE_SIZE, D), bf(D)
+        ms = timed(lambda: ops.head_prep_store(aproj, None, ctx.row_pos, None, 0, slots, ck1, cv1, 2 * nq, 2 * nkv, D, D, D,
+                                               2 * nq * D, 2 * (nq + nkv) * D - 2 * nkv * (D - V // 2), torch.bfloat16,
+                                               norm_eps=1e-6, q_norm_w=wn1, k_norm_w=wn1), flush=flush)
+        record(f"kupedra head_prep_store weighted norm {label}", ms,
+               nbytes=T * (2 * nq + 4 * nkv) * D * (4 + 2))
+        qq = bf(T, 2 * nq * hd)
+        pairs = sum(sum(min(p + i + 1, win) for i in range(n)) for p, n in zip(pos0, q_lens))
+        keys = sum(min(p + n, win + n - 1) for p, n in zip(pos0, q_lens))
+        for name, cap in (("window + cap on the scores", 50.0), ("window (difedra, without its sink)", 0.0)):
+            ms = timed(lambda: ops.attention(qq, ck, cv, ctx, ctx.groups[0], 2 * nq, nkv, hd, win, D ** -0.5, softcap=cap),
+                       flush=flush)
+            record(f"attention {name} {label}", ms, nbytes=keys * 2 * nkv * hd * 2 + 4 * T * nq * hd * 2,
+                   flops=4.0 * pairs * 2 * nq * hd)
+        attn, gproj = bf(T, 2 * nq * hd), f32(T, nq * V)
+        ms = timed(lambda: ops.map_difference(attn, nq, V, hd, 0.5, 1e-6, 0.6), flush=flush)
+        record(f"map_difference {label}", ms, nbytes=T * nq * (2 * hd + V) * 2)
+        one_map = bf(T, nq * hd)
+        ms = timed(lambda: ops.head_gate(one_map, gproj, 0, False, nq, V, hd), flush=flush)
+        record(f"ritizen head_gate {label}", ms, nbytes=T * nq * (hd * 2 + V * (4 + 2)))
+        # ---- the sums that close a sublayer
+        x, a, w1 = f32(T, width), f32(T, width), bf(width)
+        ms = timed(lambda: ops.stream_post_norm(x, a, w1, 2.0, 1e-6, copy=True), flush=flush)
+        record(f"stream_post_norm {label}", ms, nbytes=T * width * (4 + 4 + 4 + 2))
+        ms = timed(lambda: ops.stream_norm_add(x, a, w1, 1e-6, copy=True), flush=flush)
+        record(f"bukatar stream_norm_add {label}", ms, nbytes=T * width * (4 + 4 + 4 + 2))
+        # ---- the experts
+        E, ident, top, F = m["experts"], m["identity"], m["top"], m["expert_ff"]
+        logits, corr = f32(T, E + ident), 0.01 * f32(E + ident)
+        route = lambda: ops.moe_route(logits, E + ident, top, renorm=False, correction=corr, groups=m["groups"],  # noqa: E731
+                                      keep=m["keep"], scale=1.5)
+        record(f"moe_route, corrected, in groups {label}", timed(route, flush=flush), nbytes=T * ((E + ident) * 4 + top * 8))
+        ms = timed(lambda: ops.moe_route(logits, E + ident, top, renorm=False), flush=flush)
+        record(f"moe_route (kupedra) {label}", ms, nbytes=T * ((E + ident) * 4 + top * 8))
+        chosen, weight, _ = route()
+        lay = ops.moe_layout(chosen, E, torch.bfloat16, width, F)
+        y, shared = f32(lay.rows, width), f32(T, width)
+        real = int((chosen < E).sum())
+        ms = timed(lambda: ops.moe_combine_norm(x, y, lay.pos_of, weight, chosen, E, shared, None, w1, 2.0, 1e-6, copy=True),
+                   flush=flush)
+        record(f"moe_combine_norm {label}", ms, nbytes=width * 4 * real + T * width * (4 + 4 + 4 + 2))
+        ms = timed(lambda: ops.moe_combine(y, lay.pos_of, weight, shared, None), flush=flush)
+        record(f"moe_combine (kupedra) {label}", ms, nbytes=width * 4 * real + T * width * 8)
+        # ---- the token's side vector
+        n = m["side"]
+        table, p = bf(q["vocab_size"], n), f32(T, n)
+        ids = torch.randint(0, q["vocab_size"], (T,), dtype=torch.int32, device=dev)
+        ms = timed(lambda: ops.token_gate(p, table, ids, 0), flush=flush)
+        record(f"token_gate {label}", ms, nbytes=T * n * (4 + 2 + 2))
+        h = bf(T, n)
+        ms = timed(lambda: ops.gelu_tanh_(h), flush=flush)
+        record(f"ritizen gelu {label}", ms, nbytes=T * n * 4)
+    ops.take_device_errors()
+    return rows
+
+
+def run_arch_nudusun(args):
+    shape, layers = args.shape, args.layers or 4
+    pk, pk_src = peaks()
+    qcfg = dict(SHAPES[shape], num_hidden_layers=layers)
+    folders = {"nudusun": arch_folder(nudusun_config(shape, layers), f"nudusun_{shape}_L{layers}"),
+               "kupedra": arch_folder(kupedra_config(shape, layers), f"kupedra_{shape}_L{layers}"),
+               "qwen2": model_folder(SHAPES[shape], layers)}
+    clocks = ClockSampler()
+    with clocks:
+        models = {name: model_points(folder, args.batch, args.prompt_len, PREFILL_TOKENS, 20)
+                  for name, folder in folders.items()}
+        kernels = kernel_points_nudusun(shape, args.batch, args.prompt_len + 512, PREFILL_TOKENS, pk)
+    print(json.dumps({
+        "arch": "nudusun", "beside": ["kupedra", "qwen2"], "shape": shape, "layers": layers, "batch": args.batch,
+        "prompt_len": args.prompt_len, "prefill_tokens": PREFILL_TOKENS, "dtype": "bf16",
+        "data": "synthetic: random weights N(0, 0.02) seed 0", "nudusun_mixers": NUDUSUN_SHAPES[shape],
+        "hidden": qcfg["hidden_size"], "intermediate": qcfg["intermediate_size"], "vocab": qcfg["vocab_size"],
+        "models": models, "kernels": kernels, "peaks": dict(pk, source=pk_src), "clocks": clocks.summary()}))
+    return 0
+
+
 def kv_bytes_per_token(cfg, layers):
     d = cfg["hidden_size"] // cfg["num_attention_heads"]
     return 2 * layers * 2 * cfg["num_key_value_heads"] * d
@@ -1324,13 +1519,13 @@ def main() -> int:
     ap.add_argument("--stack-stamps", action="store_true",
                     help="run a few eager decode steps with the decode stack's in-kernel clock on and print what "
                          "each kind of phase took")
-    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "sogulix", "ritizen", "bukatar", "kupedra", "difedra"],
+    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "sogulix", "ritizen", "bukatar", "kupedra", "difedra", "nudusun"],
                     help="sogulix: instead of the headline run, prefill and decode throughput of the Sogulix design "
                          "beside Qwen2 at the layer sizes of --shape (0.5B or 1.5B; --layers, default 4), and each "
                          "of its kernels beside Qwen2's like kernel; prints its own line.  ritizen: the same for the "
                          "Ritizen design, beside Sogulix and Qwen2; bukatar: the same for the Bukatar design, beside "
                          "Ritizen and Qwen2; kupedra and difedra: the same for those "
-                         "designs, beside Bukatar and Qwen2")
+                         "designs, beside Bukatar and Qwen2; nudusun: the same for that design, beside Kupedra and Qwen2")
     ap.add_argument("--only-prefill", type=int, default=0, metavar="TOKENS",
                     help="run only a prefill of TOKENS tokens a few times and print its time (for profiling)")
     args = ap.parse_args()
@@ -1382,6 +1577,11 @@ def main() -> int:
             ap.error("--arch difedra knows the shapes " + ", ".join(sorted(DIFEDRA_SHAPES)))
         args.layers = 0 if args.layers == cfg["num_hidden_layers"] else args.layers
         return run_arch_difedra(args)
+    if args.arch == "nudusun":
+        if args.shape not in NUDUSUN_SHAPES:
+            ap.error("--arch nudusun knows the shapes " + ", ".join(sorted(NUDUSUN_SHAPES)))
+        args.layers = 0 if args.layers == cfg["num_hidden_layers"] else args.layers
+        return run_arch_nudusun(args)
     folder = model_folder(cfg, args.layers)
     pk, pk_src = peaks()
     if args.serve:
