@@ -225,7 +225,8 @@ def forward(cfg, w, tokens, layers_out=None, margins=None):
         x = rms_norm(alpha * x + mixer(x, w, p + "mix.", layer["mixer"], eps), w[p + "norm1"], eps)
         if layer.get("mlp") is not None:
             x = rms_norm(alpha * x + routed_experts(x, w, p + "mlp.", layer["mlp"], margins), w[p + "norm2"], eps)
-        x = x + token_input(x, w, p, tokens, i, cfg["token_side"]["dim"], eps)
+        if cfg.get("token_side") is not None:
+            x = x + token_input(x, w, p, tokens, i, cfg["token_side"]["dim"], eps)
         if layers_out is not None:
             layers_out.append(x)
     return rms_norm(x, w["final.norm"], eps) @ w["head"].T
