@@ -1370,21 +1370,21 @@ def kernel_points_nudusun(shape, batch, ctx_len, prefill_tokens, pk):
         def prepare():
             return ops.delta_prepare(proj, ch + hv, ch + hv + H, K, H, G, D, V, conv_w, hb, hb, kept, ctx, D ** -0.5, 1e-6)
 
-        dq, dk, dv, decay, rate, qk = prepare()
-        walk = lambda: ops.decay_scan(dq, dk, dv, state, ctx, H, G, D, V, a_tok=decay, s_tok=rate, c_tok=qk)  # noqa: E731
+        operands = prepare()
+        dq, dk, dv, s_tok, a_tok = f32(T, gd), f32(T, gd), operands[1], torch.rand(T, H, device=dev), torch.rand(T, H, device=dev)
+        walk = lambda: ops.delta_walk(*operands, state, ctx, H, G, D, V, proj=proj, kept=kept)  # noqa: E731
         o = walk()
         gate = proj[:, ch: ch + hv]
         finish = lambda: ops.head_norm_gate(o, gate, w_v, ctx, H, V, 1e-6)  # noqa: E731
-        prep_bytes = T * (2 * ch + 5 * H) * 4 + B * (K - 1) * ch * 8
-        walk_bytes = T * (2 * gd + 2 * hv + 3 * H) * 4 + 2 * state.numel() * 4
+        prep_bytes = T * (2 * ch + 4 * H + 7 * G) * 4 + B * (K - 1) * ch * 4
+        walk_bytes = T * (2 * gd + 2 * hv + 2 * H + 7 * G) * 4 + 2 * state.numel() * 4 + B * (K - 1) * ch * 8
         walk_flops = 6.0 * T * H * D * V if prompt else None
         record(f"delta_prepare {label}", timed(prepare, flush=flush), nbytes=prep_bytes)
         record(f"gated delta rule, the walk {label}", timed(walk, flush=flush), nbytes=walk_bytes, flops=walk_flops)
         record(f"head_norm_gate {label}", timed(finish, flush=flush), nbytes=T * hv * (4 + 4 + 2))
 
         def whole():
-            a = prepare()
-            ops.decay_scan(a[0], a[1], a[2], state, ctx, H, G, D, V, a_tok=a[3], s_tok=a[4], c_tok=a[5])
+            ops.delta_walk(*prepare(), state, ctx, H, G, D, V, proj=proj, kept=kept)
             finish()
 
         record(f"gated delta rule, all of it {label}", timed(whole, flush=flush),
@@ -1394,7 +1394,7 @@ def kernel_points_nudusun(shape, batch, ctx_len, prefill_tokens, pk):
         ms = timed(lambda: ops.delta_rule(sproj, dpre, ones, ones, ones, square, ctx, H, D, 1e-6, 0.6), flush=flush)
         record(f"sogulix delta_rule, all of it {label}", ms, nbytes=T * H * D * (6 * 4 + 2) + 2 * square.numel() * 4,
                flops=8.0 * T * H * D * D if prompt else None)
-        ms = timed(lambda: ops.decay_scan(dq, dk, dv, state, ctx, H, G, D, V, a_tok=decay, s_tok=rate), flush=flush)
+        ms = timed(lambda: ops.decay_scan(dq, dk, dv, state, ctx, H, G, D, V, a_tok=a_tok, s_tok=s_tok), flush=flush)
         record(f"ritizen decay_scan decay per token {label}", ms, nbytes=walk_bytes,
                flops=4.0 * T * H * D * V if prompt else None)
         ms = timed(lambda: ops.ssm_prepare(proj, 0, ch + hv, ch, K, H, conv_w, conv_w[:, 0].contiguous(), hb, hb, kept, ctx),

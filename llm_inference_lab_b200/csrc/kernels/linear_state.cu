@@ -2,13 +2,9 @@
 //
 //     S_t = a_t * S_{t-1} + (s_t * k_t) v_t^T,        o_t = S_t^T q_t
 //
-// or, by the delta rule, what the decayed state already holds at the key makes way for the new value:
-//
-//     S_t = a_t * S_{t-1} + k_t u_t^T,   u_t = s_t * (v_t - a_t * S_{t-1}^T k_t),   o_t = S_t^T q_t
-//
 // a_t is a constant of the head (linear attention with a fixed decay) or a number per token and head (a
-// state-space mixer, where a_t = exp(-exp(A_log) * dt_t) and s_t = dt_t; the gated delta rule, where s_t is the
-// rate of writing); q and k may be shared by the heads of a group.  The state is 32-bit, is read at a request's first row of the step and written back
+// state-space mixer, where a_t = exp(-exp(A_log) * dt_t) and s_t = dt_t); q and k may be shared by the
+// heads of a group.  The state is 32-bit, is read at a request's first row of the step and written back
 // after its last, and every product and sum of the recurrence is 32-bit, token by token in order, so a
 // position's result does not depend on how the sequence was cut into steps.
 //
@@ -18,11 +14,6 @@
 //                     before a step's first row come from the request's kept inputs) with bias and SiLU;
 //                     dt = softplus(dt + dt_bias); a = exp(-exp(A_log) * dt)
 //   ssm_keep_inputs   the request's last taps - 1 inputs of x, B, C replace the kept ones
-//   delta_prepare     for the gated delta rule, from the 32-bit input projection [q | k | v | gate | b | a]: the
-//                     causal convolution per channel of q, k, v with SiLU (the inputs kept as above), unit
-//                     vectors per q and k head, q times a constant, q . k, rate sigmoid(b), decay
-//                     exp(-exp(A_log) * softplus(a + dt_bias))
-//   head_norm_gate    every head's output over its own root mean square, a weight all heads share, SiLU(gate)
 //   gated_norm        the heads' outputs side by side (+ skip * x), a gate, an RMS norm in equal parts with
 //                     a weight, in either order (gate first with SiLU, or norm first with a sigmoid),
 //                     rounded to T for the output projection
@@ -55,37 +46,6 @@ template <int N> __device__ __forceinline__ void cp_async_wait_group() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
-// two 32-bit floats in one 64-bit register, for packed arithmetic
-typedef unsigned long long pair_t;
-__device__ __forceinline__ pair_t pair_of(float v) {
-  pair_t d;
-  asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(v));
-  return d;
-}
-__device__ __forceinline__ pair_t pair_of(float lo, float hi) {
-  pair_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ void pair_split(pair_t v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ float pair_sum(pair_t v) {
-  float lo, hi;
-  pair_split(v, lo, hi);
-  return lo + hi;
-}
-__device__ __forceinline__ pair_t pair_fma(pair_t a, pair_t b, pair_t c) {
-  pair_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ pair_t pair_mul(pair_t a, pair_t b) {
-  pair_t d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-
 struct ScanParams {
   float* out;            // [tokens, ld_o]: head h at h * V
   int ld_o;
@@ -96,7 +56,6 @@ struct ScanParams {
   int ld_v;
   const float* a_tok;    // [tokens, ld_a] decay per token and head, or null
   const float* s_tok;    // [tokens, ld_a] scale of the key per token and head, or null (1)
-  const float* c_tok;    // [tokens, ld_a] q . k per token and head (the delta rule only)
   int ld_a;
   const float* a_head;   // [H] decay per head, read when a_tok is null
   float* state;          // [slots, H, N, V]
@@ -121,11 +80,7 @@ struct ScanParams {
 // the helpers apply the SiLU to chunk c + 1, whose rows their cp.async copies have brought (16 bytes a copy
 // where the operands' addresses allow it: `vec`), and start the copies of chunk c + 2 into the buffer the
 // walkers left one chunk ago.  Three buffers, one barrier of the whole CTA per chunk.
-//
-// DELTA: the delta rule.  The output needs only the old state, o = a (q . S) + c u with c = q . k, so a token costs
-// two independent sums over a column, reduced by the same two levels of shuffles, and one multiply-add a row that
-// waits for them; the decay a S runs beside the sums.  Rows are taken two at a time (packed 32-bit multiply-adds).
-template <int R, bool DELTA>
+template <int R>
 __global__ void __launch_bounds__(256) decay_scan_kernel(ScanParams p) {
   extern __shared__ __align__(16) float smem[];
   constexpr int RS = R + 4;                      // floats between two threads' shares of a token's keys
@@ -133,7 +88,7 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(ScanParams p) {
   constexpr bool AHEAD = R <= 16;                // the next token's operands are loaded a token ahead
   pdl_trigger();
   const int walkers = blockDim.x / 2, Vs = walkers / SCAN_P;
-  const int tok_floats = 2 * NP + Vs + 4;        // k | q | v | a | s | c | (one unused, which keeps rows 16-byte aligned)
+  const int tok_floats = 2 * NP + Vs + 4;        // k | q | v | a | s | (two unused, which keep rows 16-byte aligned)
   const int h = blockIdx.y, r = blockIdx.z, g = h / (p.H / p.G);
   const bool helper = threadIdx.x >= walkers;
   const int tid = helper ? threadIdx.x - walkers : threadIdx.x;      // index within the half
@@ -188,14 +143,11 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(ScanParams p) {
         else cp_async4(dst + 2 * NP + (c - 2 * p.N), v0 + (size_t)tt * p.ld_v + (c - 2 * p.N));
       }
     }
-    if (p.a_tok != nullptr) {      // a token's decay and key scale (and q . k): one helper each
-      constexpr int SCALARS = DELTA ? 3 : 2;
-      for (int e = tid; e < SCALARS * cnt; e += walkers) {
-        const int tt = e / SCALARS, which = e - tt * SCALARS;
-        const float* src = which == 0 ? p.a_tok : which == 1 ? p.s_tok : p.c_tok;
-        if (src != nullptr)
-          cp_async4(base + tt * tok_floats + 2 * NP + Vs + which, src + (size_t)(t0 + first + tt) * p.ld_a + h);
-      }
+    if (p.a_tok != nullptr && tid < 2 * cnt) {      // a token's decay and key scale: one helper each
+      const int tt = tid >> 1, which = tid & 1;
+      const float* src = which == 0 ? p.a_tok : p.s_tok;
+      if (src != nullptr)
+        cp_async4(base + tt * tok_floats + 2 * NP + Vs + which, src + (size_t)(t0 + first + tt) * p.ld_a + h);
     }
   };
   // after the copies of `chunk` have landed for every helper: SiLU of q, k and v, once per element
@@ -231,13 +183,6 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(ScanParams p) {
     }
     if (p.a_tok == nullptr) a_const = p.a_head[h];
   }
-  pair_t S2[DELTA ? R / 2 : 1];
-  if constexpr (DELTA) {
-    if (!helper) {
-#pragma unroll
-      for (int i = 0; i < R / 2; ++i) S2[i] = pair_of(S[2 * i], S[2 * i + 1]);
-    }
-  }
   __syncthreads();
 
   for (int c = 0; c < n_chunks; ++c) {
@@ -252,62 +197,6 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(ScanParams p) {
       const int cnt = min(SCAN_CT, n_tok - c * SCAN_CT);
       const float* base = buffer(c);
       float* out = p.out + (size_t)(t0 + c * SCAN_CT) * p.ld_o + h * p.V + col;
-      if constexpr (DELTA) {
-        // the state (S2), keys and queries as pairs of neighbouring rows
-        ulonglong2 kk[R / 4], qq[R / 4];
-        float4 sc;
-        float vj;
-        auto load = [&](int tt, ulonglong2* k_to, ulonglong2* q_to, float4& s_to, float& v_to) {
-          const float* tok = base + tt * tok_floats;
-          const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(tok + part * RS);
-          const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(tok + NP + part * RS);
-#pragma unroll
-          for (int i = 0; i < R / 4; ++i) k_to[i] = k4[i], q_to[i] = q4[i];
-          s_to = *reinterpret_cast<const float4*>(tok + 2 * NP + Vs);      // a, s, q . k
-          v_to = tok[2 * NP + j];
-        };
-        if (AHEAD) load(0, kk, qq, sc, vj);
-        for (int tt = 0; tt < cnt; ++tt) {
-          ulonglong2 kn[AHEAD ? R / 4 : 1], qn[AHEAD ? R / 4 : 1];
-          float4 sn = make_float4(0.f, 0.f, 0.f, 0.f);
-          float vn = 0.f;
-          if (AHEAD) {
-            if (tt + 1 < cnt) load(tt + 1, kn, qn, sn, vn);
-          } else {
-            load(tt, kk, qq, sc, vj);
-          }
-          pair_t k0 = pair_of(0.f), k1 = pair_of(0.f), q0 = pair_of(0.f), q1 = pair_of(0.f);
-          const pair_t a2 = pair_of(sc.x);
-#pragma unroll
-          for (int i = 0; i < R / 4; ++i) {
-            k0 = pair_fma(kk[i].x, S2[2 * i], k0);
-            q0 = pair_fma(qq[i].x, S2[2 * i], q0);
-            k1 = pair_fma(kk[i].y, S2[2 * i + 1], k1);
-            q1 = pair_fma(qq[i].y, S2[2 * i + 1], q1);
-          }
-          float sk = pair_sum(k0) + pair_sum(k1), sq = pair_sum(q0) + pair_sum(q1);
-#pragma unroll
-          for (int i = 0; i < R / 2; ++i) S2[i] = pair_mul(a2, S2[i]);
-#pragma unroll
-          for (int o = 1; o < SCAN_P; o <<= 1) {
-            sk += __shfl_xor_sync(0xffffffffu, sk, o);
-            sq += __shfl_xor_sync(0xffffffffu, sq, o);
-          }
-          const float u = sc.y * fmaf(-sc.x, sk, vj);
-          const pair_t u2 = pair_of(u);
-#pragma unroll
-          for (int i = 0; i < R / 4; ++i) {
-            S2[2 * i] = pair_fma(kk[i].x, u2, S2[2 * i]);
-            S2[2 * i + 1] = pair_fma(kk[i].y, u2, S2[2 * i + 1]);
-          }
-          if (part == 0 && col < p.V) out[(size_t)tt * p.ld_o] = fmaf(sc.z, u, sc.x * sq);
-          if (AHEAD) {
-#pragma unroll
-            for (int i = 0; i < R / 4; ++i) kk[i] = kn[i], qq[i] = qn[i];
-            sc = sn, vj = vn;
-          }
-        }
-      } else {
       float4 kk[R / 4], qq[R / 4];
       float a, vj;
       auto load = [&](int tt, float4* k_to, float4* q_to, float& a_to, float& v_to) {
@@ -351,17 +240,12 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(ScanParams p) {
           a = an, vj = vn;
         }
       }
-      }
     }
     __syncthreads();
   }
   if (helper) {
     cp_async_wait_group<0>();
   } else if (p.write) {
-    if constexpr (DELTA) {
-#pragma unroll
-      for (int i = 0; i < R / 2; ++i) pair_split(S2[i], S[2 * i], S[2 * i + 1]);
-    }
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       const int n = part * R + i;
@@ -443,114 +327,6 @@ __global__ void __launch_bounds__(kThreads) ssm_keep_inputs_kernel(SsmParams p, 
   }
 }
 
-// ---- gated delta rule: convolutions, unit vectors, rates, decays -------------------------------
-// One warp per (row, unit), the eight warps of a block on eight consecutive rows of one unit (neighbouring rows
-// read the same inputs).  Units: 0 .. G - 1 the q and k head of a group, then the H value heads, then one for
-// the rates and decays of all heads.
-struct DeltaParams {
-  const float* proj;     // [tokens, ld]: q at 0 (G * D), k at G * D, v at 2 G D (H * V), rates at b_at, decays at a_at
-  int ld, b_at, a_at, taps, H, G, D, V, tokens;
-  const float* kept;     // [slots, taps - 1, 2 G D + H V]
-  const int* row_req;
-  const int* q_start;
-  const int* state_slot;
-  int n_slots;
-  float q_scale, unit_eps;
-  float* q;              // [tokens, G * D]
-  float* k;
-  float* v;              // [tokens, H * V]
-  float* decay;          // [tokens, H]
-  float* rate;
-  float* qk;
-};
-
-template <typename T>
-__global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const T* __restrict__ taps_w, const T* __restrict__ a_log,
-                                                                 const T* __restrict__ dt_bias, DeltaParams p) {
-  pdl_trigger();
-  pdl_wait();
-  constexpr int kPerLane = 8;      // heads of up to 256 key channels
-  const int lane = threadIdx.x & 31, t = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), unit = blockIdx.y;
-  if (t >= p.tokens) return;
-  const int r = p.row_req[t], first = p.q_start[r], slot = p.state_slot[r];
-  const bool padding = slot == -1;      // a row of padding leaves as zeros
-  if (!padding && (slot < 0 || slot >= p.n_slots)) {
-    if (lane == 0) lab_set_error(LAB_ERR_PAGE_RANGE);
-    return;
-  }
-  const int K = p.taps, gd = p.G * p.D, C = 2 * gd + p.H * p.V;
-  const float* kept = p.kept + (padding ? 0 : (size_t)slot * (K - 1) * C);
-  auto channel = [&](int c) {      // the convolution's output of one channel, through SiLU
-    if (padding) return 0.f;
-    float acc = 0.f;
-    for (int jj = 0; jj < K; ++jj) {
-      const int src = t - (K - 1) + jj;      // the last tap meets the row itself
-      const float u = src >= first ? p.proj[(size_t)src * p.ld + c] : kept[(size_t)((K - 1) + (src - first)) * C + c];
-      acc = fmaf(to_f32(taps_w[(size_t)c * K + jj]), u, acc);
-    }
-    return silu_f(acc);
-  };
-  if (unit < p.G) {
-    float qv[kPerLane], kv[kPerLane], qq = 0.f, kk = 0.f, qk = 0.f;
-#pragma unroll
-    for (int i = 0; i < kPerLane; ++i) {
-      const int e = lane + 32 * i;
-      qv[i] = kv[i] = 0.f;
-      if (e < p.D) qv[i] = channel(unit * p.D + e), kv[i] = channel(gd + unit * p.D + e);
-      qq = fmaf(qv[i], qv[i], qq);
-      kk = fmaf(kv[i], kv[i], kk);
-    }
-    const float q_mult = p.q_scale / sqrtf(warp_sum(qq) + p.unit_eps), k_mult = 1.0f / sqrtf(warp_sum(kk) + p.unit_eps);
-#pragma unroll
-    for (int i = 0; i < kPerLane; ++i) {
-      const int e = lane + 32 * i;
-      if (e >= p.D) break;
-      qv[i] *= q_mult, kv[i] *= k_mult;
-      qk = fmaf(qv[i], kv[i], qk);
-      p.q[(size_t)t * gd + unit * p.D + e] = qv[i];
-      p.k[(size_t)t * gd + unit * p.D + e] = kv[i];
-    }
-    qk = warp_sum(qk);
-    const int per = p.H / p.G;
-    for (int h = lane; h < per; h += 32) p.qk[(size_t)t * p.H + unit * per + h] = qk;
-  } else if (unit < p.G + p.H) {
-    const int at = (unit - p.G) * p.V;
-    for (int e = lane; e < p.V; e += 32) p.v[(size_t)t * p.H * p.V + at + e] = channel(2 * gd + at + e);
-  } else {
-    for (int h = lane; h < p.H; h += 32) {
-      const float dt = softplus_f(p.proj[(size_t)t * p.ld + p.a_at + h] + to_f32(dt_bias[h]));
-      p.decay[(size_t)t * p.H + h] = padding ? 0.f : expf(-expf(to_f32(a_log[h])) * dt);
-      p.rate[(size_t)t * p.H + h] = padding ? 0.f : sigmoid_f(p.proj[(size_t)t * p.ld + p.b_at + h]);
-    }
-  }
-}
-
-// out[t, h * V + i] = o / rms(o of head h) * w[i] * silu(gate[t, h * V + i]), rounded to T; a warp per (row, head).
-// Rows of requests without a state slot (padding) leave as zeros.
-template <typename T>
-__global__ void __launch_bounds__(kThreads) head_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ o,
-                                                                  const float* __restrict__ gate, int ld_g,
-                                                                  const T* __restrict__ w, const int* __restrict__ row_req,
-                                                                  const int* __restrict__ state_slot, int tokens, int H,
-                                                                  int V, float eps) {
-  pdl_trigger();
-  pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long unit = (long long)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
-  if (unit >= (long long)tokens * H) return;
-  const int t = (int)(unit / H), h = (int)(unit - (long long)t * H);
-  const size_t at = (size_t)t * H * V + (size_t)h * V;
-  if (state_slot[row_req[t]] == -1) {
-    for (int i = lane; i < V; i += 32) out[at + i] = from_f32<T>(0.f);
-    return;
-  }
-  float ss = 0.f;
-  for (int i = lane; i < V; i += 32) ss = fmaf(o[at + i], o[at + i], ss);
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
-  for (int i = lane; i < V; i += 32)
-    out[at + i] = from_f32<T>(o[at + i] * inv * to_f32(w[i]) * silu_f(gate[(size_t)t * ld_g + h * V + i]));
-}
-
 // ---- gate and norm of the heads' outputs ------------------------------------------------------
 // y[i] = o[t, i] + skip[head of i] * x[t, i]; gate_first: y *= silu(gate), then y / rms(part of i) * w;
 // else y / rms(part) * w * sigmoid(gate); times `mult`, rounded to T.
@@ -591,19 +367,13 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(T* __restrict__ ou
   }
 }
 
-template <int R, bool DELTA>
-int launch_scan_as(const ScanParams& p, int requests, int vs, cudaStream_t stream) {
-  const size_t smem = (size_t)3 * SCAN_CT * (2 * SCAN_P * (R + 4) + vs + 4) * sizeof(float);
-  if (smem > 48 * 1024)
-    cudaFuncSetAttribute(decay_scan_kernel<R, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  dim3 grid((p.V + vs - 1) / vs, p.H, requests);
-  return (int)lab_launch(decay_scan_kernel<R, DELTA>, grid, dim3(2 * SCAN_P * vs), smem, stream, p);
-}
-
 template <int R>
 int launch_scan(const ScanParams& p, int requests, int vs, cudaStream_t stream) {
-  return p.c_tok != nullptr ? launch_scan_as<R, true>(p, requests, vs, stream)
-                            : launch_scan_as<R, false>(p, requests, vs, stream);
+  const size_t smem = (size_t)3 * SCAN_CT * (2 * SCAN_P * (R + 4) + vs + 4) * sizeof(float);
+  if (smem > 48 * 1024)
+    cudaFuncSetAttribute(decay_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  dim3 grid((p.V + vs - 1) / vs, p.H, requests);
+  return (int)lab_launch(decay_scan_kernel<R>, grid, dim3(2 * SCAN_P * vs), smem, stream, p);
 }
 
 }  // namespace
@@ -611,20 +381,17 @@ int launch_scan(const ScanParams& p, int requests, int vs, cudaStream_t stream) 
 // Largest key size the recurrence kernel is built for.
 LAB_EXPORT int lab_decay_scan_max_keys() { return SCAN_P * 64; }
 
-// vs: columns of the state a CTA takes (8, 16 or 32).  c_tok (q . k per token and head): the delta rule, which
-// also wants a_tok and s_tok.
+// vs: columns of the state a CTA takes (8, 16 or 32).
 LAB_EXPORT int lab_decay_scan(float* out, int ld_o, const float* q, const float* k, int ld_qk, const float* v, int ld_v,
-                              const float* a_tok, const float* s_tok, const float* c_tok, int ld_a,
-                              const float* a_head, float* state,
+                              const float* a_tok, const float* s_tok, int ld_a, const float* a_head, float* state,
                               const int* q_start, const int* state_slot, int requests, int n_slots, int H, int G, int N,
                               int V, int act, int write, int vs, cudaStream_t stream) {
   if (requests <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || N <= 0 || V <= 0 || (vs != 8 && vs != 16 && vs != 32)) return (int)cudaErrorInvalidValue;
   if (a_tok == nullptr && a_head == nullptr) return (int)cudaErrorInvalidValue;
-  if (c_tok != nullptr && (a_tok == nullptr || s_tok == nullptr || act)) return (int)cudaErrorInvalidValue;
   ScanParams p;
   p.out = out; p.ld_o = ld_o; p.q = q; p.k = k; p.ld_qk = ld_qk; p.v = v; p.ld_v = ld_v; p.a_tok = a_tok;
-  p.s_tok = s_tok; p.c_tok = c_tok; p.ld_a = ld_a; p.a_head = a_head; p.state = state; p.q_start = q_start; p.state_slot = state_slot;
+  p.s_tok = s_tok; p.ld_a = ld_a; p.a_head = a_head; p.state = state; p.q_start = q_start; p.state_slot = state_slot;
   p.n_slots = n_slots; p.H = H; p.G = G; p.N = N; p.V = V; p.act = act; p.write = write;
   // 16-byte copies: every row of q, k and v, and every head's and slice's start in it, on a 16-byte boundary
   p.vec = N % 4 == 0 && V % 4 == 0 && ld_qk % 4 == 0 && ld_v % 4 == 0 &&
@@ -682,54 +449,5 @@ LAB_EXPORT int lab_gated_norm(void* out, int ld_out, const float* o, int ld_o, c
                ld_o, x, ld_x, (const __nv_bfloat16*)skip, head_size, gate, ld_g, (const __nv_bfloat16*)w, width, parts,
                gate_first, eps, mult);
   }
-  LAB_LAUNCH_CHECK();
-}
-
-// proj columns: q 0, k G * D, v 2 * G * D, rates b_at, decays a_at.  The kept inputs are read by the first kernel and
-// (with write) brought up to date by the second.
-LAB_EXPORT int lab_delta_prepare(float* q, float* k, float* v, float* decay, float* rate, float* qk, const float* proj,
-                                 int ld, int b_at, int a_at, int taps, int H, int G, int D, int V, const void* taps_w,
-                                 const void* a_log, const void* dt_bias, float* kept, const int* row_req,
-                                 const int* q_start, const int* state_slot, int tokens, int requests, int n_slots,
-                                 float q_scale, float unit_eps, int write, int dtype, cudaStream_t stream) {
-  if (tokens <= 0) return 0;
-  if (taps < 1 || H <= 0 || G <= 0 || H % G || D <= 0 || D > 256 || V <= 0) return (int)cudaErrorInvalidValue;
-  const int channels = 2 * G * D + H * V, c_blocks = (channels + kThreads - 1) / kThreads;
-  if (c_blocks > 65535 || G + H + 1 > 65535) return (int)cudaErrorInvalidValue;
-  DeltaParams p;
-  p.proj = proj; p.ld = ld; p.b_at = b_at; p.a_at = a_at; p.taps = taps; p.H = H; p.G = G; p.D = D; p.V = V;
-  p.tokens = tokens; p.kept = kept; p.row_req = row_req; p.q_start = q_start; p.state_slot = state_slot;
-  p.n_slots = n_slots; p.q_scale = q_scale; p.unit_eps = unit_eps; p.q = q; p.k = k; p.v = v; p.decay = decay;
-  p.rate = rate; p.qk = qk;
-  const dim3 grid((tokens + kThreads / 32 - 1) / (kThreads / 32), G + H + 1);
-  cudaError_t e;
-  if (dtype == LAB_F32)
-    e = lab_launch(delta_prepare_kernel<float>, grid, dim3(kThreads), 0, stream, (const float*)taps_w,
-                   (const float*)a_log, (const float*)dt_bias, p);
-  else
-    e = lab_launch(delta_prepare_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, stream, (const __nv_bfloat16*)taps_w,
-                   (const __nv_bfloat16*)a_log, (const __nv_bfloat16*)dt_bias, p);
-  if (e != cudaSuccess) return (int)e;
-  if (write && taps > 1) {
-    SsmParams s;
-    s.proj = proj; s.ld = ld; s.conv_at = 0; s.dt_at = 0; s.channels = channels; s.taps = taps; s.H = H;
-    s.kept = kept; s.row_req = row_req; s.q_start = q_start; s.state_slot = state_slot; s.n_slots = n_slots;
-    return (int)lab_launch(ssm_keep_inputs_kernel, dim3(requests, c_blocks), dim3(kThreads), 0, stream, s, requests);
-  }
-  return 0;
-}
-
-LAB_EXPORT int lab_head_norm_gate(void* out, const float* o, const float* gate, int ld_g, const void* w,
-                                  const int* row_req, const int* state_slot, int tokens, int H, int V, float eps,
-                                  int dtype, cudaStream_t stream) {
-  if (tokens <= 0) return 0;
-  const long long units = (long long)tokens * H;
-  const int blocks = (int)((units + kThreads / 32 - 1) / (kThreads / 32));
-  if (dtype == LAB_F32)
-    lab_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(kThreads), 0, stream, (float*)out, o, gate, ld_g,
-               (const float*)w, row_req, state_slot, tokens, H, V, eps);
-  else
-    lab_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(kThreads), 0, stream, (__nv_bfloat16*)out, o, gate,
-               ld_g, (const __nv_bfloat16*)w, row_req, state_slot, tokens, H, V, eps);
   LAB_LAUNCH_CHECK();
 }

@@ -1022,6 +1022,106 @@ def delta_rule(proj: torch.Tensor, decay_pre: torch.Tensor, decay_bias: torch.Te
 
 
 # ----------------------------------------------------------------------------------------
+# The gated delta rule (csrc/kernels/gated_delta.cu).
+# ----------------------------------------------------------------------------------------
+def gated_delta_supported(keys: int) -> bool:
+    return 1 <= keys <= 256
+
+
+def delta_record(keys: int) -> tuple[int, int]:
+    """(floats of a record, key channels of a share) for heads of `keys` channels: a record holds a row's k in four
+    shares with four floats of padding behind each, q likewise, then the products of q with the four keys of the row's
+    block and of k with the first three."""
+    L = lib("gated_delta")
+    return int(L.lab_delta_record_floats(keys)), int(L.lab_delta_record_share(keys))
+
+
+def delta_prepare(proj: torch.Tensor, b_at: int, a_at: int, taps: int, heads: int, groups: int, keys: int, vdim: int,
+                  taps_w: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, kept: torch.Tensor, ctx,
+                  q_scale: float, unit_eps: float):
+    """What the gated delta rule's walk reads, from the 32-bit input projection `proj`: columns [q: groups * keys
+    | k: groups * keys | v: heads * vdim] pass the causal convolution per channel (`taps_w` [channels, taps], no bias,
+    the last tap on the row itself; inputs before a request's first row of the step from `kept`
+    [slots, taps - 1, channels]) and SiLU; q and k become unit vectors per head (`unit_eps` inside the root), q times
+    `q_scale`; columns b_at and a_at on give the rates sigmoid(b) and decays exp(-exp(a_log) softplus(a + dt_bias)).
+    Returns 32-bit (records [groups, tokens, `delta_record`] of k, q and their products with the keys of the row's block
+    up to the row itself, v [tokens, heads * vdim], decay [heads, tokens], rate [heads, tokens]).  `kept` is left as it
+    is: `delta_walk` renews it."""
+    _on_gpu(proj, taps_w, a_log, dt_bias, kept)
+    tokens, channels = proj.shape[0], 2 * groups * keys + heads * vdim
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and heads % groups == 0
+    assert proj.shape[1] >= max(channels, b_at + heads, a_at + heads)
+    assert taps_w.shape == (channels, taps) and taps_w.is_contiguous() and a_log.numel() == heads
+    assert dt_bias.numel() == heads and a_log.dtype == taps_w.dtype and dt_bias.dtype == taps_w.dtype
+    assert kept.dtype == torch.float32 and kept.is_contiguous() and tuple(kept.shape[1:]) == (max(taps - 1, 0), channels)
+    if not gated_delta_supported(keys):
+        raise KernelError(f"delta_prepare: {keys} key channels are outside what the walk takes (1..256)")
+
+    def new(*shape):
+        return torch.empty(shape, dtype=torch.float32, device=proj.device)
+
+    rec, v = new(groups, tokens, delta_record(keys)[0]), new(tokens, heads * vdim)
+    decay, rate = new(heads, tokens), new(heads, tokens)
+    _check(lib("gated_delta").lab_delta_prepare(
+        _ptr(rec), _ptr(v), _ptr(decay), _ptr(rate), _ptr(proj), proj.stride(0), b_at, a_at, taps, heads, groups, keys, vdim,
+        _ptr(taps_w), _ptr(a_log), _ptr(dt_bias), _ptr(kept), _ptr(ctx.row_req), _ptr(ctx.q_start), _ptr(ctx.state_slot),
+        tokens, kept.shape[0], ctypes.c_float(q_scale), ctypes.c_float(unit_eps), dtype_code(taps_w.dtype), _stream()),
+        "delta_prepare")
+    return rec, v, decay, rate
+
+
+def delta_walk(rec: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, rate: torch.Tensor, state: torch.Tensor, ctx,
+               heads: int, groups: int, keys: int, vdim: int, write: bool = True, proj: torch.Tensor | None = None,
+               kept: torch.Tensor | None = None, shape: tuple | None = None) -> torch.Tensor:
+    """Per request and head, over the step's rows in order: S <- decay S, u = rate (v - S^T k), S <- S + k u^T, o = S^T q,
+    with S [keys, vdim] read from and (with `write`) left in `state` [slots, heads, keys, vdim]; the operands as
+    `delta_prepare` gives them, all 32-bit.  With `proj` and `kept` [slots, keep, channels] (and `write`), the request's
+    last `keep` rows of proj's first columns replace the kept ones.  `shape` (columns of the state per CTA, per thread):
+    the launch, chosen by the sizes where it is not given.  Returns o [tokens, heads * vdim]."""
+    _on_gpu(rec, v, decay, rate, state, proj, kept)
+    tokens = v.shape[0]
+    if not gated_delta_supported(keys):
+        raise KernelError(f"delta_walk: {keys} key channels are outside what the kernel takes (1..256)")
+    for t, s in ((rec, (groups, tokens, delta_record(keys)[0])), (v, (tokens, heads * vdim)), (decay, (heads, tokens)),
+                 (rate, (heads, tokens))):
+        assert t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape) == s
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, keys, vdim)
+    keep = channels = 0
+    if kept is not None and kept.shape[1] > 0:
+        keep, channels = int(kept.shape[1]), int(kept.shape[2])
+        assert kept.dtype == torch.float32 and kept.is_contiguous() and kept.shape[0] == state.shape[0]
+        assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == tokens and proj.shape[1] >= channels
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=v.device)
+    vs, cols = shape if shape is not None else delta_walk_shape(ctx.n_requests * heads, vdim)
+    _check(lib("gated_delta").lab_delta_walk(
+        _ptr(out), _ptr(rec), _ptr(v), _ptr(decay), _ptr(rate), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.state_slot), tokens,
+        ctx.n_requests, state.shape[0], heads, groups, keys, vdim, _ptr(proj if keep else None), proj.stride(0) if keep else 0,
+        _ptr(kept if keep else None), keep, channels, int(write), vs, cols, _stream()), "delta_walk")
+    return out
+
+
+def delta_walk_shape(pairs: int, vdim: int) -> tuple[int, int]:
+    """(columns of the state per CTA, per thread) of the walk over `pairs` requests and heads."""
+    return 16, 1
+
+
+def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, ctx, heads: int, vdim: int,
+                   eps: float) -> torch.Tensor:
+    """Every head of `o` [tokens, heads * vdim] (32-bit) over its own root mean square, times `weight` [vdim], times
+    silu(gate) (32-bit column slice of the same shape), rounded to the weight's storage type.  Rows of requests
+    without a state slot (padding) leave as zeros."""
+    _on_gpu(o, gate, weight)
+    tokens = o.shape[0]
+    assert o.dtype == torch.float32 and o.is_contiguous() and o.shape[1] == heads * vdim
+    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == o.shape and weight.numel() == vdim
+    out = torch.empty((tokens, heads * vdim), dtype=weight.dtype, device=o.device)
+    _check(lib("gated_delta").lab_head_norm_gate(
+        _ptr(out), _ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(ctx.row_req), _ptr(ctx.state_slot), tokens,
+        heads, vdim, ctypes.c_float(eps), dtype_code(weight.dtype), _stream()), "head_norm_gate")
+    return out
+
+
+# ----------------------------------------------------------------------------------------
 # Attention over a paged cache of latents (csrc/kernels/latent_attention.cu).
 # ----------------------------------------------------------------------------------------
 def latent_prep(proj: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, w_q: torch.Tensor, w_c: torch.Tensor,
@@ -1360,18 +1460,13 @@ def decay_scan_supported(keys: int) -> bool:
 
 def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, ctx, heads: int, groups: int,
                keys: int, vdim: int, a_head: torch.Tensor | None = None, a_tok: torch.Tensor | None = None,
-               s_tok: torch.Tensor | None = None, silu: bool = False, write: bool = True,
-               c_tok: torch.Tensor | None = None) -> torch.Tensor:
+               s_tok: torch.Tensor | None = None, silu: bool = False, write: bool = True) -> torch.Tensor:
     """Per request and head, over the step's rows in order: S <- a S + (s k) v^T, o = S^T q, with S
     [keys, vdim] read from and (with `write`) left in `state` [slots, heads, keys, vdim].  q and k are 32-bit
     column slices [tokens, groups * keys] of one tensor (same row stride), v [tokens, heads * vdim]; `a_head`
     [heads] a fixed decay per head, or `a_tok`/`s_tok` [tokens, heads] per token; `silu`: q, k and v pass a
-    SiLU first.  `c_tok` [tokens, heads], the products q . k, asks for the delta rule: S <- a S, then
-    S <- S + k u^T with u = s (v - S^T k) (`a_tok` and `s_tok` are wanted then).  Returns o [tokens, heads * vdim] in
-    32-bit."""
-    _on_gpu(q, k, v, state, a_head, a_tok, s_tok, c_tok)
-    assert c_tok is None or (a_tok is not None and s_tok is not None and not silu and c_tok.dtype == torch.float32
-                             and c_tok.shape == a_tok.shape and c_tok.stride() == a_tok.stride())
+    SiLU first.  Returns o [tokens, heads * vdim] in 32-bit."""
+    _on_gpu(q, k, v, state, a_head, a_tok, s_tok)
     tokens = v.shape[0]
     for t in (q, k, v):
         assert t.dtype == torch.float32 and t.stride(1) == 1 and t.shape[0] == tokens
@@ -1399,8 +1494,8 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
         vs = 32 if pairs * -(-vdim // 32) >= sm_count() else (16 if pairs * -(-vdim // 16) >= sm_count() else 8)
     vs = min(vs, max(8, 1 << (vdim - 1).bit_length()))
     _check(lib("linear_state").lab_decay_scan(
-        _ptr(out), out.stride(0), _ptr(q), _ptr(k), q.stride(0), _ptr(v), v.stride(0), _ptr(a_tok), _ptr(s_tok),
-        _ptr(c_tok), ld_a, _ptr(a_head), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.n_requests, state.shape[0], heads, groups,
+        _ptr(out), out.stride(0), _ptr(q), _ptr(k), q.stride(0), _ptr(v), v.stride(0), _ptr(a_tok), _ptr(s_tok), ld_a,
+        _ptr(a_head), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.state_slot), ctx.n_requests, state.shape[0], heads, groups,
         keys, vdim, int(silu), int(write), vs, _stream()), "decay_scan")
     return out
 
@@ -1429,54 +1524,6 @@ def ssm_prepare(proj: torch.Tensor, conv_at: int, dt_at: int, channels: int, tap
         tokens, ctx.n_requests, kept.shape[0], int(write), dtype_code(taps_w.dtype), _stream()), "ssm_prepare",
         2 if write and taps > 1 else 1)
     return conv, dt, decay
-
-
-def delta_prepare(proj: torch.Tensor, b_at: int, a_at: int, taps: int, heads: int, groups: int, keys: int, vdim: int,
-                  taps_w: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, kept: torch.Tensor, ctx,
-                  q_scale: float, unit_eps: float, write: bool = True):
-    """What the gated delta rule's recurrence reads, from the 32-bit input projection `proj`: columns [q: groups * keys
-    | k: groups * keys | v: heads * vdim] pass the causal convolution per channel (`taps_w` [channels, taps], no bias;
-    inputs before a request's first row of the step from `kept` [slots, taps - 1, channels], as `ssm_prepare`) and
-    SiLU; q and k become unit vectors per head (`unit_eps` inside the root), q times `q_scale`; columns b_at and a_at
-    on give the rates sigmoid(b) and decays exp(-exp(a_log) softplus(a + dt_bias)).  Returns 32-bit (q, k, v, decay,
-    rate, q . k per head)."""
-    _on_gpu(proj, taps_w, a_log, dt_bias, kept)
-    tokens, gd, hv = proj.shape[0], groups * keys, heads * vdim
-    channels = 2 * gd + hv
-    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and heads % groups == 0
-    assert proj.shape[1] >= max(channels, b_at + heads, a_at + heads)
-    assert taps_w.shape == (channels, taps) and taps_w.is_contiguous() and a_log.numel() == heads
-    assert dt_bias.numel() == heads and a_log.dtype == taps_w.dtype and dt_bias.dtype == taps_w.dtype
-    assert kept.dtype == torch.float32 and kept.is_contiguous() and tuple(kept.shape[1:]) == (max(taps - 1, 0), channels)
-    if not decay_scan_supported(keys):
-        raise KernelError(f"delta_prepare: {keys} key channels are outside what the recurrence kernel takes (1..256)")
-
-    def new(width):
-        return torch.empty((tokens, width), dtype=torch.float32, device=proj.device)
-
-    q, k, v, decay, rate, qk = new(gd), new(gd), new(hv), new(heads), new(heads), new(heads)
-    _check(lib("linear_state").lab_delta_prepare(
-        _ptr(q), _ptr(k), _ptr(v), _ptr(decay), _ptr(rate), _ptr(qk), _ptr(proj), proj.stride(0), b_at, a_at, taps, heads,
-        groups, keys, vdim, _ptr(taps_w), _ptr(a_log), _ptr(dt_bias), _ptr(kept), _ptr(ctx.row_req), _ptr(ctx.q_start),
-        _ptr(ctx.state_slot), tokens, ctx.n_requests, kept.shape[0], ctypes.c_float(q_scale), ctypes.c_float(unit_eps),
-        int(write), dtype_code(taps_w.dtype), _stream()), "delta_prepare", 2 if write and taps > 1 else 1)
-    return q, k, v, decay, rate, qk
-
-
-def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, ctx, heads: int, vdim: int,
-                   eps: float) -> torch.Tensor:
-    """Every head of `o` [tokens, heads * vdim] (32-bit) over its own root mean square, times `weight` [vdim], times
-    silu(gate) (32-bit column slice of the same shape), rounded to the weight's storage type.  Rows of requests
-    without a state slot (padding) leave as zeros."""
-    _on_gpu(o, gate, weight)
-    tokens = o.shape[0]
-    assert o.dtype == torch.float32 and o.is_contiguous() and o.shape[1] == heads * vdim
-    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == o.shape and weight.numel() == vdim
-    out = torch.empty((tokens, heads * vdim), dtype=weight.dtype, device=o.device)
-    _check(lib("linear_state").lab_head_norm_gate(
-        _ptr(out), _ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(ctx.row_req), _ptr(ctx.state_slot), tokens,
-        heads, vdim, ctypes.c_float(eps), dtype_code(weight.dtype), _stream()), "head_norm_gate")
-    return out
 
 
 def gated_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, parts: int = 1,

@@ -89,8 +89,8 @@ class GatedDelta(Mixer):
     fixed-size states (`CacheParts`).
 
     The matrices that read h are one product, taken in 32-bit; one kernel convolves, forms the unit vectors, rates
-    and decays, one walks the state (`ops.decay_scan`), one norms and gates.  All of it is 32-bit up to the rounding
-    before W_o."""
+    and decays, one walks the state in blocks of four tokens and renews the kept inputs, one norms and gates
+    (`csrc/kernels/gated_delta.cu`).  All of it is 32-bit up to the rounding before W_o."""
     decode_graph_safe = True
     CONVOLVED = ("q", "k", "v")
 
@@ -118,7 +118,7 @@ class GatedDelta(Mixer):
 
     @classmethod
     def libraries(cls, spec, dtype):
-        return [("linear_state", {})]
+        return [("gated_delta", {})]
 
     def __init__(self, spec, weights, dtype, device):
         super().__init__(spec, weights, dtype, device)
@@ -126,7 +126,7 @@ class GatedDelta(Mixer):
             int(spec[k]) for k in ("heads", "kv_heads", "dim", "vdim", "taps"))
         if self.heads % self.groups:
             raise ValueError("gated_delta: heads must be a multiple of kv_heads")
-        if not ops.decay_scan_supported(self.dim):
+        if not ops.gated_delta_supported(self.dim):
             raise ValueError(f"gated_delta: {self.dim} key channels are outside what the recurrence kernel takes")
         self.eps, self.unit_eps = float(spec["eps"]), float(spec.get("unit_eps", 1e-6))
         w = lambda n: self._weight(weights, n)  # noqa: E731
@@ -142,11 +142,11 @@ class GatedDelta(Mixer):
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
         proj = ops.linear(x, self.w_in, None, out_f32=True)
         state, kept = cache.part(0), cache.part(1)
-        q, k, v, decay, rate, qk = ops.delta_prepare(
+        operands = ops.delta_prepare(
             proj, self.rate_at, self.decay_at, self.taps, self.heads, self.groups, self.dim, self.vdim, self.conv_w,
-            self.a_log, self.dt_bias, kept.state, ctx, self.dim ** -0.5, self.unit_eps, write=cache.write)
-        o = ops.decay_scan(q, k, v, state.state, ctx, self.heads, self.groups, self.dim, self.vdim, a_tok=decay,
-                           s_tok=rate, c_tok=qk, write=cache.write)
+            self.a_log, self.dt_bias, kept.state, ctx, self.dim ** -0.5, self.unit_eps)
+        o = ops.delta_walk(*operands, state.state, ctx, self.heads, self.groups, self.dim, self.vdim, write=cache.write,
+                           proj=proj, kept=kept.state)
         y = ops.head_norm_gate(o, proj[:, self.gate_at: self.gate_at + self.hv], self.norm_weight, ctx, self.heads,
                                self.vdim, self.eps)
         return ops.linear(y, self.w_o, None, out_f32=True, allow_partial=True)

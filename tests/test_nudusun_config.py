@@ -43,7 +43,7 @@ def test_blueprint_caches_and_groups():
     assert bp.layers[0].ffn["groups"] == (3, 2) and bp.layers[0].ffn["identity"] == 3 and not bp.layers[0].ffn["renorm"]
     assert bp.layers[1].ffn["groups"] is None and bp.layers[1].ffn["shared_ff"] == 0 and bp.layers[2].ffn is None
     assert [s.block_spec["side"]["at"] for s in bp.layers] == [0, 10, 20, 30]
-    assert ("linear_state", {}) in kernel_libraries(bp, torch.bfloat16)
+    assert ("gated_delta", {}) in kernel_libraries(bp, torch.bfloat16)
     # two keys of 80 do not fit the tensor-core kernels' head: each map is a head of its own
     arch, typed = _resolve(SMALL["D"][0])
     needs = cache_plan(arch.blueprint(typed)).needs

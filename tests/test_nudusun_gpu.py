@@ -46,87 +46,120 @@ def _dtypes():
 # ---------------------------------------------------------------------------------------------
 # the gated delta rule
 # ---------------------------------------------------------------------------------------------
+def _dots(q, k, q_start):
+    """The products of every row's q and k [T, G, D] with the keys of its block of four packed rows, as far as they are
+    the request's own: [T, G, 8]."""
+    T, G, _ = q.shape
+    out = np.zeros((T, G, 8))
+    for r in range(len(q_start) - 1):
+        for t in range(q_start[r], q_start[r + 1]):
+            for j in range(max(t // 4 * 4, q_start[r]), t + 1):
+                out[t, :, j % 4] = (q[t] * k[j]).sum(-1)
+                if j < t:
+                    out[t, :, 4 + j % 4] = (k[t] * k[j]).sum(-1)
+    return out
+
+
+def _records(q, k, q_start):
+    """The rows' records [G, T, floats]: k in four shares with four zeros behind each, q likewise, the products."""
+    from llm_inference_lab_b200.kernels import ops
+    T, G, D = q.shape
+    floats, share = ops.delta_record(D)
+    assert floats == 8 * (share + 4) + 8 and 4 * share >= D
+    out = np.zeros((G, T, floats))
+    for e in range(D):
+        at = e // share * (share + 4) + e % share
+        out[:, :, at], out[:, :, 4 * (share + 4) + at] = k[:, :, e].T, q[:, :, e].T
+    out[:, :, -8:] = _dots(q, k, q_start).transpose(1, 0, 2)
+    return out
+
+
+def _walk(q, k, v, decay, rate, state, lens, slots, **more):
+    """`ops.delta_walk` over rows of q, k [T, G, D], v [T, H, V]: [T, H, V]."""
+    from llm_inference_lab_b200.kernels import ops
+    (T, G, D), (_, H, V) = q.shape, v.shape
+    ctx, _ = make_ctx(lens, [0] * len(lens), slots, page_size=64)
+    rec = _records(q, k, np.concatenate([[0], np.cumsum(lens)]))
+    return _np(ops.delta_walk(_t(rec), _t(v.reshape(T, -1)), _t(decay.T), _t(rate.T), state, ctx, H, G, D, V, **more)).reshape(T, H, V)
+
+
 @pytest.mark.parametrize("H,G,D,V", [(4, 2, 16, 24), (3, 3, 5, 7), (2, 1, 64, 64), (6, 2, 100, 33), (2, 2, 128, 40), (3, 1, 250, 16),
                                      (1, 1, 1, 1), (2, 1, 48, 130), (1, 1, 12, 8)])
 def test_delta_rule_walk(H, G, D, V):
-    """The recurrence from random states over portions of unequal length, a request of padding between them; then the
-    same rows one at a time; the states left behind.  Decays from almost nothing to almost one."""
-    torch = _torch()
+    """The recurrence from random states over portions of unequal length that start anywhere in a block of four rows, a
+    request of padding between them; then the same rows one at a time; the states left behind; every shape of launch.
+    Decays from almost nothing to almost one."""
     from llm_inference_lab_b200.kernels import ops
     rng = np.random.default_rng(D + V)
-    q_lens, slots = [37, 1, 4, 2, 16, 65], [3, 0, -1, 5, 1, 6]
-    T = sum(q_lens)
+    lens, slots = [37, 1, 4, 2, 16, 65], [3, 0, -1, 5, 1, 6]
+    T = sum(lens)
     q, k = rng.standard_normal((T, G, D)), pn.unit(rng.standard_normal((T, G, D)))
     v = rng.standard_normal((T, H, V))
-    decay, rate = rng.random((T, H)) ** 0.2, rng.random((T, H))
-    qk = np.repeat((q * k).sum(-1), H // G, axis=1)
+    decay, rate = rng.random((T, H)) ** rng.choice([0.05, 1.0, 9.0], (T, H)), rng.random((T, H))
     start = rng.standard_normal((8, H, D, V))
     want, want_state = np.zeros((T, H, V)), start.copy()
     at = 0
-    for n, slot in zip(q_lens, slots):
+    for n, slot in zip(lens, slots):
         for h in range(H):
             if slot >= 0:
                 rows, g = slice(at, at + n), h // (H // G)
                 want[rows, h], want_state[slot, h] = pn.gated_delta_rule(q[rows, g], k[rows, g], v[rows, h], decay[rows, h],
                                                                          rate[rows, h], start[slot, h])
         at += n
-    flat = lambda a: _t(a.reshape(T, -1))  # noqa: E731
-
-    def run(state, lens, where, rows, write=True):
-        ctx, _ = make_ctx(lens, [0] * len(lens), where, page_size=64)
-        a = [flat(x)[rows].contiguous() for x in (q, k, v)]
-        s = [_t(x)[rows].contiguous() for x in (decay, rate, qk)]
-        return _np(ops.decay_scan(*a, state, ctx, H, G, D, V, a_tok=s[0], s_tok=s[1], c_tok=s[2], write=write)).reshape(-1, H, V)
-
-    real = np.concatenate([np.full(n, slot >= 0) for n, slot in zip(q_lens, slots)])
-    state = _t(start)
-    got = run(state, q_lens, slots, slice(None), write=False)
-    assert np.array_equal(_np(state), _np(_t(start)))       # a call that only reads leaves the state alone
+    real = np.concatenate([np.full(n, slot >= 0) for n, slot in zip(lens, slots)])
     tol = 3e-5 * max(1.0, np.abs(want).max())
+    state_tol = 3e-5 * max(1.0, np.abs(want_state).max())
+    state = _t(start)
+    got = _walk(q, k, v, decay, rate, state, lens, slots, write=False)
+    assert np.array_equal(_np(state), _np(_t(start)))       # a call that only reads leaves the state alone
     assert np.abs(got[real] - want[real]).max() < tol
-    assert np.array_equal(run(state, q_lens, slots, slice(None))[real], got[real])
-    assert np.abs(_np(state) - want_state).max() < 3e-5 * max(1.0, np.abs(want_state).max())
+    for shape in (None, (8, 1), (16, 1), (16, 2), (24, 1), (32, 1), (32, 2), (64, 2)):
+        if D > 128 and shape is not None and shape[1] == 2:
+            continue
+        state = _t(start)
+        assert np.abs(_walk(q, k, v, decay, rate, state, lens, slots, shape=shape)[real] - want[real]).max() < tol, shape
+        assert np.abs(_np(state) - want_state).max() < state_tol, shape
     state, at = _t(start), 0
-    for n, slot in zip(q_lens, slots):
+    for n, slot in zip(lens, slots):
         for t in range(at, at + n if slot >= 0 else at):
-            assert np.abs(run(state, [1], [slot], slice(t, t + 1))[0] - want[t]).max() < tol
+            r = slice(t, t + 1)
+            assert np.abs(_walk(q[r], k[r], v[r], decay[r], rate[r], state, [1], [slot])[0] - want[t]).max() < tol
         at += n
-    assert np.abs(_np(state) - want_state).max() < 3e-5 * max(1.0, np.abs(want_state).max())
+    assert np.abs(_np(state) - want_state).max() < state_tol
     ops.take_device_errors()
 
 
 def test_delta_rule_replaces_a_far_write():
     """A value written at a key stays readable hundreds of tokens later while other keys are written and nothing decays,
-    and is gone after a write at the same key: prompt, portions of two and single tokens."""
+    and is gone after a write at the same key: prompt, portions of two and of seven, single tokens; also where the two
+    writes fall into one block."""
     from llm_inference_lab_b200.kernels import ops
-    D, V, T = 32, 8, 300
-    rng = np.random.default_rng(0)
-    basis = np.eye(D)
-    k = basis[rng.integers(1, D, size=T)]
-    v = rng.standard_normal((T, V))
-    k[3] = basis[0]
-    k[250] = basis[0]
-    q = np.tile(basis[0], (T, 1))
-    one = np.ones((T, 1))
-    qk = (q * k).sum(-1, keepdims=True)
-    want, _ = pn.gated_delta_rule(q, k, v, one[:, 0], one[:, 0])
-    assert np.allclose(want[3:250], v[3]) and np.allclose(want[250:], v[250])
-    for sizes in ((T,), (2,) * (T // 2), (1,) * T):
-        state, at, outs = _t(np.zeros((1, 1, D, V))), 0, []
-        for n in sizes:
-            ctx, _ = make_ctx([n], [at], [0], page_size=64)
-            r = slice(at, at + n)
-            outs.append(_np(ops.decay_scan(_t(q[r]), _t(k[r]), _t(v[r]), state, ctx, 1, 1, D, V, a_tok=_t(one[r]), s_tok=_t(one[r]),
-                                           c_tok=_t(qk[r]))))
-            at += n
-        assert np.abs(np.concatenate(outs) - want).max() < 1e-5
+    D, V, T = 32, 8, 308
+    for first, second in ((3, 250), (100, 103), (101, 102), (103, 104)):
+        rng = np.random.default_rng(first)
+        basis = np.eye(D)
+        k = basis[rng.integers(1, D, size=T)]
+        v = rng.standard_normal((T, V))
+        k[first] = k[second] = basis[0]
+        q = np.tile(basis[0], (T, 1))
+        one = np.ones((T, 1))
+        want, _ = pn.gated_delta_rule(q, k, v, one[:, 0], one[:, 0])
+        assert np.allclose(want[first:second], v[first]) and np.allclose(want[second:], v[second])
+        for sizes in ((T,), (2,) * (T // 2), (7,) * (T // 7), (1,) * T):
+            state, at, outs = _t(np.zeros((1, 1, D, V))), 0, []
+            for n in sizes:
+                r = slice(at, at + n)
+                outs.append(_walk(q[r, None], k[r, None], v[r, None], one[r], one[r], state, [n], [0])[:, 0])
+                at += n
+            assert np.abs(np.concatenate(outs) - want).max() < 1e-5
     ops.take_device_errors()
 
 
 @pytest.mark.parametrize("H,G,D,V,taps", [(4, 2, 16, 24, 4), (3, 1, 5, 7, 1), (2, 2, 130, 9, 7), (5, 5, 1, 3, 2), (2, 1, 256, 40, 3)])
 def test_delta_preparation(H, G, D, V, taps):
     """Convolutions across steps (portions shorter than the taps among them), unit vectors, rates and decays, the
-    products q . k; a row of padding gives zeros and leaves every slot's inputs alone."""
+    products with the keys of a row's block; a row of padding gives zeros; the kept inputs, renewed by the walk, and
+    every other slot's left alone."""
     torch = _torch()
     from llm_inference_lab_b200.kernels import ops
     rng = np.random.default_rng(D)
@@ -141,25 +174,32 @@ def test_delta_preparation(H, G, D, V, taps):
         for x in u:
             y = pn.silu(pn.causal_conv(x[:, :ch], _np(w)))
             qn, kn = pn.unit(y[:, :gd].reshape(T, G, D)) * 0.3, pn.unit(y[:, gd: 2 * gd].reshape(T, G, D))
-            want.append((qn.reshape(T, gd), kn.reshape(T, gd), y[:, 2 * gd:],
+            want.append((qn, kn, y[:, 2 * gd:],
                          np.exp(-np.exp(_np(a_log)) * pn.softplus(x[:, a_at: a_at + H] + _np(bias))),
-                         pn.sigmoid(x[:, b_at: b_at + H]), np.repeat((qn * kn).sum(-1), H // G, axis=1)))
+                         pn.sigmoid(x[:, b_at: b_at + H])))
         kept = torch.zeros((4, max(taps - 1, 0), ch), device="cuda")
+        state = torch.zeros((4, H, D, V), device="cuda")
         at = [0, 0]
         for n0, n1 in ((3, 1), (1, 2), (2, 9), (11, 1), (1, 5), (12, 12)):
             lens = [n0, 2, n1]
             ctx, _ = make_ctx(lens, [at[0], 0, at[1]], [2, -1, 0], page_size=64)
             proj = _t(np.concatenate([u[0][at[0]: at[0] + n0], 9.0 * np.ones((2, a_at + H)), u[1][at[1]: at[1] + n1]]))
             got = ops.delta_prepare(proj, b_at, a_at, taps, H, G, D, V, w, a_log, bias, kept, ctx, 0.3, 1e-6)
-            for i, name in enumerate(("q", "k", "v", "decay", "rate", "qk")):
-                g = _np(got[i])
-                assert np.abs(g[:n0] - want[0][i][at[0]: at[0] + n0]).max() < 2e-5, name
-                assert np.abs(g[n0 + 2:] - want[1][i][at[1]: at[1] + n1]).max() < 2e-5, name
-                assert not g[n0: n0 + 2].any(), name
+            q, k, v, decay, rate = (np.concatenate([want[0][i][at[0]: at[0] + n0], np.zeros_like(want[0][i][:2]),
+                                                    want[1][i][at[1]: at[1] + n1]]) for i in range(5))
+            rec = _records(q, k, [0, n0, n0 + 2, n0 + 2 + n1])
+            for name, g, w_ in (("records", got[0], rec), ("v", got[1], v), ("decay", got[2], decay.T), ("rate", got[3], rate.T)):
+                g = _np(g)
+                if name == "records":
+                    g[..., -1] = 0.0      # unused
+                assert np.abs(g - w_).max() < 2e-5, name
+            ops.delta_walk(*got, state, ctx, H, G, D, V, proj=proj, kept=kept, write=False)      # reads only
+            ops.delta_walk(*got, state, ctx, H, G, D, V, proj=proj, kept=kept)
             at = [at[0] + n0, at[1] + n1]
-        if taps > 1:
-            assert not kept[1].any() and not kept[3].any()
-            assert np.allclose(_np(kept[2]), _np(_t(u[0][T - taps + 1: T, :ch])))
+            for slot, x, n in ((2, u[0], at[0]), (0, u[1], at[1])):
+                last = np.concatenate([np.zeros((taps, ch)), _np(_t(x[:n, :ch]))])[len(x[:n]) + 1:] if taps > 1 else np.zeros((0, ch))
+                assert np.array_equal(_np(kept[slot]), last)
+        assert not kept[1].any() and not kept[3].any()
     ops.take_device_errors()
 
 
