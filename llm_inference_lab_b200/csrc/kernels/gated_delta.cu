@@ -36,7 +36,7 @@ constexpr int kThreads = 256;
 constexpr int PARTS = 4;        // threads that share one column of the state
 constexpr int BLK = 4;          // rows of a block
 constexpr int CT = 16;          // rows staged per chunk
-constexpr int HELPERS = 128;    // threads that copy chunks ahead and form the blocks' coefficients
+constexpr int HELPERS = 64;     // threads that copy chunks ahead and form the blocks' coefficients
 constexpr int DOTS = 8;         // q . k_0..3, k . k_0..2 of a row's block, one unused
 // coefficients of a block: rates, rates times G, three rows of the substitution, four of the outputs, g_3j, G
 // A record: k in PARTS shares of R channels with four floats of padding behind each (zeros beyond the head's

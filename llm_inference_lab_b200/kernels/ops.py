@@ -1092,7 +1092,7 @@ def delta_walk(rec: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, rate: to
         assert kept.dtype == torch.float32 and kept.is_contiguous() and kept.shape[0] == state.shape[0]
         assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == tokens and proj.shape[1] >= channels
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=v.device)
-    vs, cols = shape if shape is not None else delta_walk_shape(ctx.n_requests * heads, vdim)
+    vs, cols = shape if shape is not None else delta_walk_shape(ctx.n_requests * heads, keys, vdim, ctx.max_q_len)
     _check(lib("gated_delta").lab_delta_walk(
         _ptr(out), _ptr(rec), _ptr(v), _ptr(decay), _ptr(rate), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.state_slot), tokens,
         ctx.n_requests, state.shape[0], heads, groups, keys, vdim, _ptr(proj if keep else None), proj.stride(0) if keep else 0,
@@ -1100,9 +1100,23 @@ def delta_walk(rec: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, rate: to
     return out
 
 
-def delta_walk_shape(pairs: int, vdim: int) -> tuple[int, int]:
-    """(columns of the state per CTA, per thread) of the walk over `pairs` requests and heads."""
-    return 16, 1
+def delta_walk_shape(pairs: int, keys: int, vdim: int, max_q_len: int) -> tuple[int, int]:
+    """(columns of the state per CTA, per thread) of the walk over `pairs` requests and heads.  Measured for 14 to 128
+    pairs of 64 x 64 and 128 x 128 states: over a portion of a prompt the walk is one dependent chain per CTA, shortest
+    with a column a thread in slices of 16, while the CTAs find an SM each; beyond that wider slices, then two columns a
+    thread, stage the keys and queries less often.  A step of single tokens only reads and writes the state."""
+    if max_q_len == 1:
+        vs, cols = 32, 2
+    elif pairs * -(-vdim // 16) <= sm_count():
+        vs, cols = 16, 1
+    elif pairs * -(-vdim // 32) <= sm_count():
+        vs, cols = 32, 1
+    else:
+        vs, cols = 64, 2
+    if keys > 128:          # a thread's share of two columns would not fit its registers
+        vs, cols = min(vs, 32), 1
+    step = 8 * cols
+    return min(vs, -(-vdim // step) * step), cols
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, ctx, heads: int, vdim: int,
