@@ -111,8 +111,9 @@ struct PrepareParams {
 
 // One warp per (row, unit), the eight warps of a CTA on eight consecutive rows (two blocks) of one unit; neighbouring
 // rows read the same inputs.  Units: 0 .. G - 1 the q and k head of a group, then the H value heads, then one for the
-// rates and decays of all heads.  A row of padding (state slot -1) leaves as zeros.
-template <typename T>
+// rates and decays of all heads.  A row of padding (state slot -1) leaves as zeros.  TAPS: the number of taps where the
+// kernel is built for it (a channel's inputs are then all in flight at once), 0: p.taps.
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const T* __restrict__ taps_w, const T* __restrict__ a_log,
                                                                  const T* __restrict__ dt_bias, PrepareParams p) {
   extern __shared__ float keys[];      // [8][D]: the rows' unit keys (q and k units)
@@ -128,15 +129,23 @@ __global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const T* __rest
     if (lane == 0) lab_set_error(LAB_ERR_PAGE_RANGE);
     live = false;
   }
-  const int K = p.taps, gd = p.G * p.D, C = 2 * gd + p.H * p.V;
+  const int K = TAPS > 0 ? TAPS : p.taps, gd = p.G * p.D, C = 2 * gd + p.H * p.V;
   const float* kept = p.kept + (padding ? 0 : (size_t)slot * (K - 1) * C);
   auto channel = [&](int c) {      // the convolution's output of one channel, through SiLU
     if (padding || !live) return 0.f;
+    auto input = [&](int jj) {      // the last tap meets the row itself
+      const int src = t - (K - 1) + jj;
+      return src >= first ? p.proj[(size_t)src * p.ld + c] : kept[(size_t)((K - 1) + (src - first)) * C + c];
+    };
     float acc = 0.f;
-    for (int jj = 0; jj < K; ++jj) {
-      const int src = t - (K - 1) + jj;      // the last tap meets the row itself
-      const float u = src >= first ? p.proj[(size_t)src * p.ld + c] : kept[(size_t)((K - 1) + (src - first)) * C + c];
-      acc = fmaf(to_f32(taps_w[(size_t)c * K + jj]), u, acc);
+    if constexpr (TAPS > 0) {
+      float u[TAPS], w[TAPS];
+#pragma unroll
+      for (int jj = 0; jj < TAPS; ++jj) u[jj] = input(jj), w[jj] = to_f32(taps_w[(size_t)c * TAPS + jj]);
+#pragma unroll
+      for (int jj = 0; jj < TAPS; ++jj) acc = fmaf(w[jj], u[jj], acc);
+    } else {
+      for (int jj = 0; jj < K; ++jj) acc = fmaf(to_f32(taps_w[(size_t)c * K + jj]), input(jj), acc);
     }
     return silu_f(acc);
   };
@@ -481,11 +490,32 @@ __global__ void __launch_bounds__(kThreads) head_norm_gate_kernel(T* __restrict_
     for (int i = lane; i < V; i += 32) out[at + i] = from_f32<T>(0.f);
     return;
   }
-  float ss = 0.f;
-  for (int i = lane; i < V; i += 32) ss = fmaf(o[at + i], o[at + i], ss);
+  // up to 128 entries a head wait in registers, outputs, gates and weights all asked for at once
+  constexpr int kPerLane = 4;
+  const float* g = gate + (size_t)t * ld_g + h * V;
+  float y[kPerLane], z[kPerLane], ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kPerLane; ++j) {
+    const int i = lane + 32 * j;
+    y[j] = i < V ? o[at + i] : 0.f;
+    z[j] = i < V ? silu_f(g[i]) * to_f32(w[i]) : 0.f;
+    ss = fmaf(y[j], y[j], ss);
+  }
+  for (int i = lane + 32 * kPerLane; i < V; i += 32) ss = fmaf(o[at + i], o[at + i], ss);
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
-  for (int i = lane; i < V; i += 32)
-    out[at + i] = from_f32<T>(o[at + i] * inv * to_f32(w[i]) * silu_f(gate[(size_t)t * ld_g + h * V + i]));
+#pragma unroll
+  for (int j = 0; j < kPerLane; ++j) {
+    const int i = lane + 32 * j;
+    if (i < V) out[at + i] = from_f32<T>(y[j] * inv * z[j]);
+  }
+  for (int i = lane + 32 * kPerLane; i < V; i += 32) out[at + i] = from_f32<T>(o[at + i] * inv * (silu_f(g[i]) * to_f32(w[i])));
+}
+
+template <typename T>
+void launch_prepare(const PrepareParams& p, dim3 grid, size_t smem, const void* taps_w, const void* a_log, const void* dt_bias,
+                    cudaStream_t stream) {
+  auto kernel = p.taps == 4 ? delta_prepare_kernel<T, 4> : p.taps == 3 ? delta_prepare_kernel<T, 3> : delta_prepare_kernel<T, 0>;
+  lab_launch(kernel, grid, dim3(kThreads), smem, stream, (const T*)taps_w, (const T*)a_log, (const T*)dt_bias, p);
 }
 
 template <int R, int NC>
@@ -525,12 +555,8 @@ LAB_EXPORT int lab_delta_prepare(float* rec, float* v, float* decay, float* rate
   p.decay = decay; p.rate = rate;
   const dim3 grid((tokens + kThreads / 32 - 1) / (kThreads / 32), G + H + 1);
   const size_t smem = (size_t)(kThreads / 32) * D * sizeof(float);
-  if (dtype == LAB_F32)
-    lab_launch(delta_prepare_kernel<float>, grid, dim3(kThreads), smem, stream, (const float*)taps_w, (const float*)a_log,
-               (const float*)dt_bias, p);
-  else
-    lab_launch(delta_prepare_kernel<__nv_bfloat16>, grid, dim3(kThreads), smem, stream, (const __nv_bfloat16*)taps_w,
-               (const __nv_bfloat16*)a_log, (const __nv_bfloat16*)dt_bias, p);
+  if (dtype == LAB_F32) launch_prepare<float>(p, grid, smem, taps_w, a_log, dt_bias, stream);
+  else launch_prepare<__nv_bfloat16>(p, grid, smem, taps_w, a_log, dt_bias, stream);
   LAB_LAUNCH_CHECK();
 }
 

@@ -254,14 +254,22 @@ __global__ void __launch_bounds__(1024) moe_combine_norm_kernel(float* __restric
                                                                 const T* __restrict__ w, int top, int width, float alpha,
                                                                 float eps) {
   __shared__ float scratch[32];
-  extern __shared__ __align__(16) float row[];      // [width]: the sum
+  extern __shared__ __align__(16) float row[];      // [width]: the sum; then the token's places and weights [top] each
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const size_t base = (size_t)t * width;
-  const int* pos = pos_of + (size_t)t * top;
-  const float* wt = weight != nullptr ? weight + (size_t)t * top : nullptr;
-  const float keep = alpha + identity_weight(chosen + (size_t)t * top, wt, top, identity_from);
+  // the token's choice is read once, side by side: every later load depends on it
+  int* pos = reinterpret_cast<int*>(row + (width + 3) / 4 * 4);
+  float* wt = reinterpret_cast<float*>(pos + top);
+  float id_w = 0.f;
+  for (int k = threadIdx.x; k < top; k += blockDim.x) {
+    const float c = weight != nullptr ? weight[(size_t)t * top + k] : 1.f;
+    pos[k] = pos_of[(size_t)t * top + k];
+    wt[k] = c;
+    if (chosen[(size_t)t * top + k] >= identity_from) id_w += c;
+  }
+  const float keep = alpha + block_sum(id_w, scratch);      // (its barriers also publish the places and weights)
   const float gs = shared_gate != nullptr ? shared_gate[t] : 1.f;
   float ss = 0.f;
   if constexpr (VEC) {
@@ -270,11 +278,12 @@ __global__ void __launch_bounds__(1024) moe_combine_norm_kernel(float* __restric
       auto add = [&](float c, float4 v) {
         acc = make_float4(fmaf(c, v.x, acc.x), fmaf(c, v.y, acc.y), fmaf(c, v.z, acc.z), fmaf(c, v.w, acc.w));
       };
-#pragma unroll 2
+      const float4 own = load4(x + base + i);
+#pragma unroll 4
       for (int k = 0; k < top; ++k)
-        if (pos[k] >= 0) add(wt != nullptr ? wt[k] : 1.f, load4(y + (size_t)pos[k] * width + i));
+        if (pos[k] >= 0) add(wt[k], load4(y + (size_t)pos[k] * width + i));
       if (shared != nullptr) add(gs, sum_splits4(shared, shared_splits, split_stride, base + i));
-      add(keep, load4(x + base + i));
+      add(keep, own);
       store4(row + i, acc);
       ss += acc.x * acc.x + acc.y * acc.y + acc.z * acc.z + acc.w * acc.w;
     }
@@ -282,7 +291,7 @@ __global__ void __launch_bounds__(1024) moe_combine_norm_kernel(float* __restric
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
       float acc = 0.f;
       for (int k = 0; k < top; ++k)
-        if (pos[k] >= 0) acc = fmaf(wt != nullptr ? wt[k] : 1.f, y[(size_t)pos[k] * width + i], acc);
+        if (pos[k] >= 0) acc = fmaf(wt[k], y[(size_t)pos[k] * width + i], acc);
       if (shared != nullptr) {
         float sum = 0.f;
         for (int s = 0; s < shared_splits; ++s) sum += shared[(size_t)s * split_stride + base + i];
@@ -315,7 +324,7 @@ template <typename T>
 int launch_combine_norm(float* x, void* copy, const float* y, const int* pos_of, const float* weight, const int* chosen,
                         int identity_from, const float* shared, int shared_splits, const float* shared_gate, const void* w,
                         int tokens, int top, int width, float alpha, float eps, cudaStream_t stream) {
-  const size_t smem = (size_t)width * sizeof(float);
+  const size_t smem = ((size_t)(width + 3) / 4 * 4 + 2 * top) * sizeof(float);
   auto on16 = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
   const bool vec = width % 4 == 0 && on16(x) && on16(copy) && on16(y) && on16(shared) && on16(w);
   auto kernel = vec ? moe_combine_norm_kernel<T, true> : moe_combine_norm_kernel<T, false>;

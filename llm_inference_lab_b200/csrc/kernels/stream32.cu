@@ -219,19 +219,52 @@ __global__ void __launch_bounds__(kThreads) embed_position_kernel(float* __restr
 // order; x[t] += y / rms(y) * w; and (if asked) the new x[t] rounded to T, for the product that reads
 // the stream next, or, with `w_next`, the new x[t] normed once more: x[t] / rms(x[t]) * w_next, rounded (the
 // norm that opens the next sublayer, in the same pass).
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(1024) stream_norm_add_kernel(float* __restrict__ x, T* __restrict__ copy,
                                                                const float* __restrict__ a, int a_splits,
                                                                long long split_stride, const T* __restrict__ bias,
                                                                const T* __restrict__ w, int hidden, float eps,
                                                                const T* __restrict__ w_next) {
   __shared__ float scratch[32];
-  extern __shared__ float row[];      // [hidden]: the product's row, summed once
+  extern __shared__ __align__(16) float row[];      // [hidden]: the product's row, summed once
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const size_t base = (size_t)t * hidden;
   float ss = 0.f;
+  if constexpr (VEC) {      // rows of whole groups of four
+    for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
+      float4 v = sum_splits4(a, a_splits, split_stride, base + i);
+      if (bias != nullptr) {
+        const float4 b = load4(bias + i);
+        v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+      }
+      store4(row + i, v);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+    float s2 = 0.f;
+    for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
+      const float4 p = load4(row + i), g = load4(w + i), o = load4(x + base + i);
+      const float4 v = make_float4(o.x + p.x * inv * g.x, o.y + p.y * inv * g.y, o.z + p.z * inv * g.z, o.w + p.w * inv * g.w);
+      store4(x + base + i, v);
+      if (w_next != nullptr) {
+        store4(row + i, v);
+        s2 += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      } else if (copy != nullptr) {
+        store4(copy + base + i, v);
+      }
+    }
+    if (w_next == nullptr || copy == nullptr) return;
+    s2 = block_sum(s2, scratch);
+    const float inv2 = 1.0f / sqrtf(s2 / (float)hidden + eps);
+    for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
+      const float4 v = load4(row + i), g = load4(w_next + i);
+      store4(copy + base + i, make_float4(v.x * inv2 * g.x, v.y * inv2 * g.y, v.z * inv2 * g.z, v.w * inv2 * g.w));
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float v = sum_splits(a, a_splits, split_stride, base + i);
     if (bias != nullptr) v += to_f32(bias[i]);
@@ -450,27 +483,28 @@ LAB_EXPORT int lab_embed_position(float* out, const void* table, const void* pos
   LAB_LAUNCH_CHECK();
 }
 
+template <typename T>
+static int launch_norm_add(float* x, void* copy, const float* a, int a_splits, const void* bias, const void* w, int tokens,
+                           int hidden, float eps, const void* w_next, cudaStream_t stream) {
+  const size_t smem = (size_t)hidden * sizeof(float);
+  auto on16 = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
+  const bool vec = hidden % 4 == 0 && on16(x) && on16(copy) && on16(a) && on16(bias) && on16(w) && on16(w_next);
+  auto kernel = vec ? stream_norm_add_kernel<T, true> : stream_norm_add_kernel<T, false>;
+  const int per = vec ? hidden / 4 : hidden;
+  const int threads = tokens <= 64 || per < kThreads ? (per >= 1024 ? 1024 : (per + 31) / 32 * 32) : kThreads;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  return (int)lab_launch(kernel, dim3(tokens), dim3(threads), smem, stream, x, (T*)copy, a, a_splits,
+                         (long long)tokens * hidden, (const T*)bias, (const T*)w, hidden, eps, (const T*)w_next);
+}
+
 LAB_EXPORT int lab_stream_norm_add(float* x, void* copy, const float* a, int a_splits, const void* bias, const void* w,
                                    int tokens, int hidden, float eps, const void* w_next, int dtype,
                                    cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  const long long stride = (long long)tokens * hidden;
-  const size_t smem = (size_t)hidden * sizeof(float);
-  if (smem > 160 * 1024) return (int)cudaErrorInvalidValue;
-  const int threads = tokens <= 64 ? (hidden >= 1024 ? 1024 : (hidden + 31) / 32 * 32) : kThreads;
-  if (dtype == LAB_F32) {
-    if (smem > 48 * 1024)
-      cudaFuncSetAttribute(stream_norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    lab_launch(stream_norm_add_kernel<float>, dim3(tokens), dim3(threads), smem, stream, x, (float*)copy, a, a_splits,
-               stride, (const float*)bias, (const float*)w, hidden, eps, (const float*)w_next);
-  } else {
-    if (smem > 48 * 1024)
-      cudaFuncSetAttribute(stream_norm_add_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    lab_launch(stream_norm_add_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), smem, stream, x, (__nv_bfloat16*)copy,
-               a, a_splits, stride, (const __nv_bfloat16*)bias, (const __nv_bfloat16*)w, hidden, eps,
-               (const __nv_bfloat16*)w_next);
-  }
-  LAB_LAUNCH_CHECK();
+  if ((size_t)hidden * sizeof(float) > 160 * 1024) return (int)cudaErrorInvalidValue;
+  if (dtype == LAB_F32)
+    return launch_norm_add<float>(x, copy, a, a_splits, bias, w, tokens, hidden, eps, w_next, stream);
+  return launch_norm_add<__nv_bfloat16>(x, copy, a, a_splits, bias, w, tokens, hidden, eps, w_next, stream);
 }
 
 LAB_EXPORT int lab_stream_round(void* out, const float* x, long long n, int dtype, cudaStream_t stream) {
@@ -514,7 +548,7 @@ static int launch_post_norm(float* x, void* copy, const float* a, int a_splits, 
   auto on16 = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
   const bool vec = hidden % 4 == 0 && on16(x) && on16(copy) && on16(a) && on16(w);
   auto kernel = vec ? stream_post_norm_kernel<T, true> : stream_post_norm_kernel<T, false>;
-  const int per = vec ? (hidden + 3) / 4 : hidden;
+  const int per = vec ? hidden / 4 : hidden;
   const int threads = tokens <= 64 || per < kThreads ? (per >= 1024 ? 1024 : (per + 31) / 32 * 32) : kThreads;
   if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   return (int)lab_launch(kernel, dim3(tokens), dim3(threads), smem, stream, x, (T*)copy, a, a_splits,

@@ -57,3 +57,15 @@ def test_prefill_tiles_are_always_a_shape_the_kernels_take():
         if splits > 1:
             assert -(-K // 64) // splits >= 16, "a split with too few k-tiles"
             assert -(-T // 128) * -(-n_out // bn) * splits <= ops.sm_count()
+
+
+def test_delta_walk_shapes_are_what_the_kernel_takes():
+    """Slices of whole warps of walkers, two columns a thread only where registers allow, narrow slices while every CTA
+    finds an SM of its own, and no slice far beyond the state's columns."""
+    for pairs, keys, vdim, q_len in itertools.product((1, 14, 56, 128, 2000), (1, 16, 64, 128, 129, 256), (1, 8, 24, 64, 128, 200),
+                                                      (1, 2, 2048)):
+        vs, cols = ops.delta_walk_shape(pairs, keys, vdim, q_len)
+        assert cols in (1, 2) and vs % (8 * cols) == 0 and 0 < vs <= 32 * cols and vs < vdim + 8 * cols
+        assert cols == 1 or keys <= 128
+    assert ops.delta_walk_shape(14, 64, 64, 2048) == (16, 1) and ops.delta_walk_shape(56, 64, 64, 512) == (32, 1)
+    assert ops.delta_walk_shape(128, 128, 128, 512) == (64, 2) and ops.delta_walk_shape(14, 64, 64, 1) == (32, 2)
