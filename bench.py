@@ -1424,13 +1424,13 @@ def kernel_points_nudusun(shape, batch, ctx_len, prefill_tokens, pk):
         pairs = sum(sum(min(p + i + 1, win) for i in range(n)) for p, n in zip(pos0, q_lens))
         keys = sum(min(p + n, win + n - 1) for p, n in zip(pos0, q_lens))
         for name, cap in (("window + cap on the scores", 50.0), ("window (difedra, without its sink)", 0.0)):
-            ms = timed(lambda: ops.attention(qq, ck, cv, ctx, ctx.groups[0], 2 * nq, nkv, hd, win, D ** -0.5, softcap=cap),
-                       flush=flush)
-            record(f"attention {name} {label}", ms, nbytes=keys * 2 * nkv * hd * 2 + 4 * T * nq * hd * 2,
+            ms = timed(lambda: ops.attention(qq, ck, cv, ctx, ctx.groups[0], 2 * nq, nkv, hd, win, D ** -0.5, softcap=cap,
+                                             out_f32=cap > 0.0), flush=flush)
+            record(f"attention {name} {label}", ms, nbytes=keys * 2 * nkv * hd * 2 + 2 * T * nq * hd * (6 if cap > 0.0 else 4),
                    flops=4.0 * pairs * 2 * nq * hd)
-        attn, gproj = bf(T, 2 * nq * hd), f32(T, nq * V)
-        ms = timed(lambda: ops.map_difference(attn, nq, V, hd, 0.5, 1e-6, 0.6), flush=flush)
-        record(f"map_difference {label}", ms, nbytes=T * nq * (2 * hd + V) * 2)
+        attn, gproj = f32(T, 2 * nq * hd), f32(T, nq * V)
+        ms = timed(lambda: ops.map_difference(attn, nq, V, hd, 0.5, 1e-6, 0.6, dtype=torch.bfloat16), flush=flush)
+        record(f"map_difference {label}", ms, nbytes=T * nq * (2 * hd * 4 + V * 2))
         one_map = bf(T, nq * hd)
         ms = timed(lambda: ops.head_gate(one_map, gproj, 0, False, nq, V, hd), flush=flush)
         record(f"ritizen head_gate {label}", ms, nbytes=T * nq * (hd * 2 + V * (4 + 2)))

@@ -44,6 +44,16 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// One output, or two neighbours, of an attention kernel: rounded to bfloat16, or (f32) as they are.
+__device__ __forceinline__ void store_out(void* out, size_t at, float v, int f32) {
+  if (f32) reinterpret_cast<float*>(out)[at] = v;
+  else reinterpret_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(v);
+}
+__device__ __forceinline__ void store_out2(void* out, size_t at, float lo, float hi, int f32) {
+  if (f32) *reinterpret_cast<float2*>(reinterpret_cast<float*>(out) + at) = make_float2(lo, hi);
+  else *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(out) + at) = pack_bf16(lo, hi);
+}
+
 // Where key `j` of a request lies: element offset of its row in the cache, -1 if its page was
 // given back, -2 if the block table names a page outside the pool (reported by the caller).
 __device__ __forceinline__ long long key_offset(const int* __restrict__ bt, int j, int kvh, int n_kv, int page_size,

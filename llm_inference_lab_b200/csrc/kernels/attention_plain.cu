@@ -18,7 +18,7 @@
 // added to the softmax's denominator, a key with score 0 and no value; with `sinks`, a number per query head,
 // exp(sinks[h]) instead), and `dist_bias` [n_q, bias_len]: a number per head and distance query - key that is
 // added to the scaled score, distances from bias_len - 1 on sharing the last entry.  `softcap` c > 0: the scaled score
-// s becomes c * tanh(s / c) first.
+// s becomes c * tanh(s / c) first.  `out_f32`: the output is 32-bit whatever T is.
 #include "common.cuh"
 
 namespace {
@@ -27,11 +27,11 @@ constexpr int MAX_DPL = 8;  // dims per lane: head sizes up to 256
 
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32) attention_plain_kernel(
-    T* __restrict__ out, int out_stride, const T* __restrict__ q, int q_stride, const T* __restrict__ cache_k,
+    void* __restrict__ out, int out_stride, const T* __restrict__ q, int q_stride, const T* __restrict__ cache_k,
     const T* __restrict__ cache_v, const int* __restrict__ row_req, const int* __restrict__ row_pos,
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int d, int page_size, int num_pages,
     int window, float scale, int keep_first, int sink, const float* __restrict__ sinks,
-    const float* __restrict__ dist_bias, int bias_len, float softcap) {
+    const float* __restrict__ dist_bias, int bias_len, float softcap, int out_f32) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
@@ -119,7 +119,10 @@ __global__ void __launch_bounds__(WARPS * 32) attention_plain_kernel(
       num += wt * part[w * (d + 2) + i];
       den += wt * part[w * (d + 2) + d + 1];
     }
-    out[(size_t)t * out_stride + (size_t)h * d + i] = from_f32<T>(den > 0.f ? num / den : 0.f);
+    const size_t at = (size_t)t * out_stride + (size_t)h * d + i;
+    const float o = den > 0.f ? num / den : 0.f;
+    if (out_f32) reinterpret_cast<float*>(out)[at] = o;
+    else reinterpret_cast<T*>(out)[at] = from_f32<T>(o);
   }
 }
 }  // namespace
@@ -128,7 +131,7 @@ LAB_EXPORT int lab_attention_plain(void* out, int out_stride, const void* q, int
                                    const void* cache_v, const int* row_req, const int* row_pos, const int* block_table,
                                    int max_blocks, int tokens, int n_q, int n_kv, int d, int page_size, int num_pages,
                                    int window, float scale, int keep_first, int sink, const float* sinks,
-                                   const float* dist_bias, int bias_len, float softcap, int dtype,
+                                   const float* dist_bias, int bias_len, float softcap, int out_f32, int dtype,
                                    cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (d > 32 * MAX_DPL || d <= 0 || n_q % n_kv || (dist_bias != nullptr && bias_len < 1)) return (int)cudaErrorInvalidValue;
@@ -136,13 +139,13 @@ LAB_EXPORT int lab_attention_plain(void* out, int out_stride, const void* q, int
   dim3 grid(tokens, n_q);
   const size_t smem = (size_t)(d + WARPS * (d + 2)) * sizeof(float);
   if (dtype == LAB_F32)
-    return (int)lab_launch(attention_plain_kernel<float>, grid, dim3(WARPS * 32), smem, stream, (float*)out, out_stride,
+    return (int)lab_launch(attention_plain_kernel<float>, grid, dim3(WARPS * 32), smem, stream, out, out_stride,
                            (const float*)q, q_stride, (const float*)cache_k, (const float*)cache_v, row_req, row_pos,
                            block_table, max_blocks, n_q, n_kv, d, page_size, num_pages, window, scale, keep_first,
-                           sink, sinks, dist_bias, bias_len, softcap);
+                           sink, sinks, dist_bias, bias_len, softcap, out_f32);
   return (int)lab_launch(attention_plain_kernel<__nv_bfloat16>, grid, dim3(WARPS * 32), smem, stream,
-                         (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
+                         out, out_stride, (const __nv_bfloat16*)q, q_stride,
                          (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v, row_req, row_pos, block_table,
                          max_blocks, n_q, n_kv, d, page_size, num_pages, window, scale, keep_first, sink, sinks, dist_bias,
-                         bias_len, softcap);
+                         bias_len, softcap, out_f32);
 }

@@ -28,12 +28,12 @@ constexpr int PF_TILE_BYTES = PF_BN * ROW_BYTES;
 constexpr int PF_SMEM = PF_BM * ROW_BYTES + 4 * PF_TILE_BYTES;  // Q + 2 stages of (K, V)
 
 __global__ void __launch_bounds__(PF_THREADS) attention_prefill_kernel(
-    __nv_bfloat16* __restrict__ out, int out_stride, const __nv_bfloat16* __restrict__ q, int q_stride,
+    void* __restrict__ out, int out_stride, const __nv_bfloat16* __restrict__ q, int q_stride,
     const __nv_bfloat16* __restrict__ cache_k, const __nv_bfloat16* __restrict__ cache_v,
     const int* __restrict__ q_start, const int* __restrict__ kv_len_arr, const int* __restrict__ pos0_arr,
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window,
     float scale_log2, int min_q_len, const float* __restrict__ sink, int keep, const float* __restrict__ dist_bias,
-    int bias_len, float cap_log2, float arg_log2) {
+    int bias_len, float cap_log2, float arg_log2, int out_f32) {
   extern __shared__ __align__(16) uint8_t smem[];
   pdl_trigger();
   pdl_wait();
@@ -143,10 +143,9 @@ __global__ void __launch_bounds__(PF_THREADS) attention_prefill_kernel(
     const int row = r0 + warp * 16 + (lane >> 2) + 8 * r;
     if (row >= ql) continue;
     const float inv = l[r] > 0.f ? 1.f / l[r] : 0.f;
-    __nv_bfloat16* dst = out + (size_t)(qs + row) * out_stride + (size_t)h * D + 2 * (lane & 3);
+    const size_t dst = (size_t)(qs + row) * out_stride + (size_t)h * D + 2 * (lane & 3);
 #pragma unroll
-    for (int t = 0; t < DTILES; ++t)
-      *reinterpret_cast<uint32_t*>(dst + t * 8) = pack_bf16(o[t][2 * r] * inv, o[t][2 * r + 1] * inv);
+    for (int t = 0; t < DTILES; ++t) store_out2(out, dst + t * 8, o[t][2 * r] * inv, o[t][2 * r + 1] * inv, out_f32);
   }
 }
 
@@ -193,12 +192,12 @@ struct DcLayout {
 // one cluster barrier everyone finds all it needs at home: no scratch and no merge kernel.
 template <bool CLUSTER = false>
 __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
-    __nv_bfloat16* __restrict__ out, int out_stride, const __nv_bfloat16* __restrict__ q, int q_stride,
+    void* __restrict__ out, int out_stride, const __nv_bfloat16* __restrict__ q, int q_stride,
     __nv_bfloat16* __restrict__ cache_k, __nv_bfloat16* __restrict__ cache_v,
     const int* __restrict__ q_start, const int* __restrict__ kv_len_arr, const int* __restrict__ block_table,
     int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window, float scale_log2, int splits,
     float* __restrict__ part_acc, float* __restrict__ part_ml, int keep, const float* __restrict__ sink,
-    const float* __restrict__ dist_bias, int bias_len, float cap_log2, float arg_log2) {
+    const float* __restrict__ dist_bias, int bias_len, float cap_log2, float arg_log2, int out_f32) {
   extern __shared__ __align__(16) uint8_t smem[];
   using L = DcLayout<CLUSTER>;
   pdl_trigger();
@@ -357,7 +356,7 @@ __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
     }
     const int head = head0 + row;
     if (splits == 1) {
-      out[(size_t)qs * out_stride + (size_t)head * D + dim] = __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+      store_out(out, (size_t)qs * out_stride + (size_t)head * D + dim, den > 0.f ? num / den : 0.f, out_f32);
     } else if constexpr (CLUSTER) {
       // to the CTA that merges element i: slot `split` of its receive area
       const int share = (n_heads * D + splits - 1) / splits;
@@ -398,17 +397,17 @@ __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
           num += wt * from[i - lo_item];
           den += wt * from[share + 2 * row + 1];
         }
-        out[(size_t)qs * out_stride + (size_t)(head0 + row) * D + dim] =
-            __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+        store_out(out, (size_t)qs * out_stride + (size_t)(head0 + row) * D + dim, den > 0.f ? num / den : 0.f, out_f32);
       }
     }
   }
 }
 
 // Merge of the splits: one block per (request, query head), D threads.
-__global__ void attention_merge_kernel(__nv_bfloat16* __restrict__ out, int out_stride,
+__global__ void attention_merge_kernel(void* __restrict__ out, int out_stride,
                                        const int* __restrict__ q_start, int n_q, int splits,
-                                       const float* __restrict__ part_acc, const float* __restrict__ part_ml) {
+                                       const float* __restrict__ part_acc, const float* __restrict__ part_ml,
+                                       int out_f32) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x, head = blockIdx.y, dim = threadIdx.x;
@@ -442,7 +441,7 @@ __global__ void attention_merge_kernel(__nv_bfloat16* __restrict__ out, int out_
       }
     }
   }
-  out[(size_t)qs * out_stride + (size_t)head * D + dim] = __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+  store_out(out, (size_t)qs * out_stride + (size_t)head * D + dim, den > 0.f ? num / den : 0.f, out_f32);
 }
 
 }  // namespace
@@ -462,13 +461,14 @@ LAB_EXPORT long long lab_attention_decode_scratch_floats(int requests, int n_q, 
 static float cap_of(float softcap) { return softcap > 0.f ? softcap * LOG2E : 0.f; }
 static float cap_arg(float softcap, float scale) { return softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f; }
 
-// softcap c > 0: the scaled score s becomes c * tanh(s / c), before a bias by distance.
+// softcap c > 0: the scaled score s becomes c * tanh(s / c), before a bias by distance.  out_f32: the output is 32-bit
+// (out_stride in its elements) and is not rounded.
 LAB_EXPORT int lab_attention_prefill(void* out, int out_stride, const void* q, int q_stride, const void* cache_k,
                                      const void* cache_v, const int* q_start, const int* kv_len, const int* pos0,
                                      const int* block_table, int max_blocks, int requests, int max_q_len, int n_q,
                                      int n_kv, int page_size, int num_pages, int window, float scale, int min_q_len,
                                      const float* sink, int keep_first, const float* dist_bias, int bias_len,
-                                     float softcap, cudaStream_t stream) {
+                                     float softcap, int out_f32, cudaStream_t stream) {
   if (requests <= 0 || max_q_len <= 0) return 0;
   if (n_q % n_kv || q_stride % 8 || (((uintptr_t)q) & 15)) return (int)cudaErrorInvalidValue;
   static bool configured = false;
@@ -479,11 +479,11 @@ LAB_EXPORT int lab_attention_prefill(void* out, int out_stride, const void* q, i
   }
   dim3 grid((max_q_len + PF_BM - 1) / PF_BM, n_q, requests);
   return (int)lab_launch(attention_prefill_kernel, grid, dim3(PF_THREADS), (size_t)PF_SMEM, stream,
-                         (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
+                         out, out_stride, (const __nv_bfloat16*)q, q_stride,
                          (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v, q_start, kv_len, pos0,
                          block_table, max_blocks, n_q, n_kv, page_size, num_pages, window, scale * LOG2E, min_q_len,
                          sink, window > 0 && keep_first > 0 ? keep_first : 0, dist_bias, dist_bias != nullptr ? bias_len : 0,
-                         cap_of(softcap), cap_arg(softcap, scale));
+                         cap_of(softcap), cap_arg(softcap, scale), out_f32);
 }
 
 static int decode_launch(void* out, int out_stride, const void* q, int q_stride, const void* cache_k,
@@ -491,7 +491,7 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
                          int max_blocks, int requests, int n_q, int n_kv, int page_size, int num_pages, int window,
                          float scale, int splits, float* scratch, bool may_cluster, cudaStream_t stream,
                          int keep_first = 0, const float* sink = nullptr, const float* dist_bias = nullptr,
-                         int bias_len = 0, float softcap = 0.f) {
+                         int bias_len = 0, float softcap = 0.f, int out_f32 = 0) {
   if (requests <= 0) return 0;
   if (dist_bias == nullptr) bias_len = 0;
   const int keep = window > 0 && keep_first > 0 ? keep_first : 0;
@@ -527,23 +527,24 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = g_lab_pdl ? 2 : 1;
-    return (int)cudaLaunchKernelEx(&cfg, attention_decode_kernel<true>, (__nv_bfloat16*)out, out_stride,
+    return (int)cudaLaunchKernelEx(&cfg, attention_decode_kernel<true>, out, out_stride,
                                    (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v,
                                    q_start, kv_len, block_table, max_blocks, n_q, n_kv, page_size, num_pages, window,
                                    scale * LOG2E, splits, (float*)nullptr, (float*)nullptr, keep, sink, dist_bias,
-                                   bias_len, cap_of(softcap), cap_arg(softcap, scale));
+                                   bias_len, cap_of(softcap), cap_arg(softcap, scale), out_f32);
   }
   float* part_acc = scratch;
   float* part_ml = scratch ? scratch + (size_t)requests * n_q * splits * D : nullptr;
   cudaError_t e = lab_launch(attention_decode_kernel<false>, grid, dim3(DC_THREADS), (size_t)DcLayout<false>::SMEM, stream,
-                             (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride,
+                             out, out_stride, (const __nv_bfloat16*)q, q_stride,
                              (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v, q_start, kv_len, block_table,
                              max_blocks, n_q, n_kv, page_size, num_pages, window, scale * LOG2E, splits, part_acc,
-                             part_ml, keep, sink, dist_bias, bias_len, cap_of(softcap), cap_arg(softcap, scale));
+                             part_ml, keep, sink, dist_bias, bias_len, cap_of(softcap), cap_arg(softcap, scale),
+                             out_f32);
   if (e != cudaSuccess) return (int)e;
   if (splits > 1)
-    e = lab_launch(attention_merge_kernel, dim3(requests, n_q), dim3(D), 0, stream, (__nv_bfloat16*)out, out_stride,
-                   q_start, n_q, splits, (const float*)part_acc, (const float*)part_ml);
+    e = lab_launch(attention_merge_kernel, dim3(requests, n_q), dim3(D), 0, stream, out, out_stride,
+                   q_start, n_q, splits, (const float*)part_acc, (const float*)part_ml, out_f32);
   return (int)e;
 }
 
@@ -553,16 +554,16 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
 // keep_first: beside a window, the first that many positions stay visible; sink: null or a number per
 // query head that joins the softmax's denominator as exp(sink); dist_bias: null or [n_q, bias_len] floats, a
 // number per head and distance query - key added to the scaled score (distances from bias_len - 1 on share the
-// last entry); softcap: as lab_attention_prefill.
+// last entry); softcap, out_f32: as lab_attention_prefill.
 LAB_EXPORT int lab_attention_decode(void* out, int out_stride, const void* q, int q_stride, const void* cache_k,
                                     const void* cache_v, const int* q_start, const int* kv_len,
                                     const int* block_table, int max_blocks, int requests, int n_q, int n_kv,
                                     int page_size, int num_pages, int window, float scale, int splits, float* scratch,
                                     int cluster_merge, int keep_first, const float* sink, const float* dist_bias,
-                                    int bias_len, float softcap, cudaStream_t stream) {
+                                    int bias_len, float softcap, int out_f32, cudaStream_t stream) {
   return decode_launch(out, out_stride, q, q_stride, cache_k, cache_v, q_start, kv_len, block_table, max_blocks,
                        requests, n_q, n_kv, page_size, num_pages, window, scale, splits, scratch, cluster_merge != 0,
-                       stream, keep_first, sink, dist_bias, bias_len, softcap);
+                       stream, keep_first, sink, dist_bias, bias_len, softcap, out_f32);
 }
 
 // ----------------------------------------------------------------------------------------

@@ -82,12 +82,12 @@ struct Barriers {
 
 __global__ void __launch_bounds__(THREADS) attention_prefill_tc05_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-    const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, int out_stride,
+    const __grid_constant__ CUtensorMap map_v, void* __restrict__ out, int out_stride,
     const __nv_bfloat16* __restrict__ cache_k, const __nv_bfloat16* __restrict__ cache_v,
     const int* __restrict__ q_start, const int* __restrict__ kv_len_arr, const int* __restrict__ pos0_arr,
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window,
     float scale_log2, int min_q_len, int keep, const float* __restrict__ sink, const float* __restrict__ dist_bias,
-    int bias_len, float bias_mult, float cap_log2, float arg_log2) {
+    int bias_len, float bias_mult, float cap_log2, float arg_log2, int out_f32) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   Barriers* bar = reinterpret_cast<Barriers*>(smem + OFF_BAR);
@@ -413,13 +413,22 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc05_kernel(
       if (ok) {
         tc_fence_after();
         const float inv = l > 0.f ? 1.f / l : 0.f;
-        __nv_bfloat16* dst = out + (size_t)(qs + r0 + row) * out_stride + (size_t)h * D;
+        const size_t at = (size_t)(qs + r0 + row) * out_stride + (size_t)h * D;
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + at;
 #pragma unroll
         for (int part = 0; part < D / 32; ++part) {
           uint32_t r[32];
           tmem_ld32_issue(o_addr + part * 32, r);   // every lane takes part in the load
           tmem_wait();
           if (!row_valid || n_tiles == 0) continue;
+          if (out_f32) {      // (the host checks that 16-byte stores are aligned)
+            float* d32 = reinterpret_cast<float*>(out) + at + part * 32;
+#pragma unroll
+            for (int q4 = 0; q4 < 8; ++q4)
+              store4(d32 + 4 * q4, make_float4(__uint_as_float(r[4 * q4]) * inv, __uint_as_float(r[4 * q4 + 1]) * inv,
+                                               __uint_as_float(r[4 * q4 + 2]) * inv, __uint_as_float(r[4 * q4 + 3]) * inv));
+            continue;
+          }
 #pragma unroll
           for (int q8 = 0; q8 < 4; ++q8) {
             const uint4 packed = make_uint4(
@@ -462,17 +471,19 @@ LAB_EXPORT int lab_attention_tc05_supports(int page_size) {
 // query head that joins the softmax's denominator as exp(sink); dist_bias: null or [n_q, bias_len] floats
 // (bias_len up to lab_attention_tc05_bias_max()), a number per head and distance query - key added to the scaled
 // score, distances from bias_len - 1 on sharing the last entry.  softcap c > 0: the scaled score s becomes
-// c * tanh(s / c), before the bias.
+// c * tanh(s / c), before the bias.  out_f32: the output is 32-bit (out_stride in its elements) and is not rounded.
 LAB_EXPORT int lab_attention_tc05_bias_max() { return BIAS_MAX; }
 LAB_EXPORT int lab_attention_prefill_tc05(void* out, int out_stride, const void* q, int q_stride, int total_rows,
                                           const void* cache_k, const void* cache_v, const int* q_start,
                                           const int* kv_len, const int* pos0, const int* block_table, int max_blocks,
                                           int requests, int max_q_len, int n_q, int n_kv, int page_size, int num_pages,
                                           int window, float scale, int min_q_len, int keep_first, const float* sink,
-                                          const float* dist_bias, int bias_len, float softcap, cudaStream_t stream) {
+                                          const float* dist_bias, int bias_len, float softcap, int out_f32,
+                                          cudaStream_t stream) {
   if (requests <= 0 || max_q_len <= 0) return 0;
   if (dist_bias == nullptr) bias_len = 0;
   if (bias_len < 0 || bias_len > BIAS_MAX || !(scale > 0.f)) return (int)cudaErrorInvalidValue;
+  if (out_f32 && (out_stride % 4 || (((uintptr_t)out) & 15))) return (int)cudaErrorInvalidValue;
   if (!lab_attention_tc05_supports(page_size) || n_q % n_kv || q_stride % 8 || (((uintptr_t)q) & 15) ||
       (((uintptr_t)cache_k) & 15) || (((uintptr_t)cache_v) & 15))
     return (int)cudaErrorInvalidValue;
@@ -491,9 +502,9 @@ LAB_EXPORT int lab_attention_prefill_tc05(void* out, int out_stride, const void*
   }
   dim3 grid(n_q, (max_q_len + BM - 1) / BM, requests);
   return (int)lab_launch(attention_prefill_tc05_kernel, grid, dim3(THREADS), (size_t)SMEM, stream, mq, mk, mv,
-                         (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v,
+                         out, out_stride, (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v,
                          q_start, kv_len, pos0, block_table, max_blocks, n_q, n_kv, page_size, num_pages, window,
                          softcap > 0.f ? 1.f : scale * LOG2E, min_q_len, window > 0 && keep_first > 0 ? keep_first : 0, sink,
                          dist_bias, bias_len, softcap > 0.f ? LOG2E : 1.0f / scale, softcap > 0.f ? softcap * LOG2E : 0.f,
-                         softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f);
+                         softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f, out_f32);
 }

@@ -284,11 +284,12 @@ __global__ void __launch_bounds__(kThreads) head_gate_kernel(T* __restrict__ out
 }
 
 // Two score maps over the same values, combined: a1 - lambda * a2 over its root mean square within the head (V
-// entries, eps inside the root), times `mult`, rounded to T and packed for the output projection.  A head's two
+// entries, eps inside the root), times `mult`, rounded to T and packed for the output projection.  A is how the maps'
+// outputs are stored: where lambda is near 1 the difference of two alike maps is small next to their own rounding.  A head's two
 // maps lie at heads 2 h and 2 h + 1 of attn (grouped 0) or, with the queries ordered (group, map, head in the group),
 // at (2 (h / per) + m) per + h % per (grouped 1, per = heads of a group).  A warp per (row, head).
-template <typename T>
-__global__ void __launch_bounds__(kThreads) map_difference_kernel(T* __restrict__ out, const T* __restrict__ attn, int ld_a,
+template <typename T, typename A>
+__global__ void __launch_bounds__(kThreads) map_difference_kernel(T* __restrict__ out, const A* __restrict__ attn, int ld_a,
                                                                   int tokens, int H, int V, int HD, int grouped, int per,
                                                                   float lambda, float eps, float mult) {
   pdl_trigger();
@@ -298,8 +299,8 @@ __global__ void __launch_bounds__(kThreads) map_difference_kernel(T* __restrict_
   if (unit >= (long long)tokens * H) return;
   const int t = (int)(unit / H), h = (int)(unit - (long long)t * H);
   const int h1 = grouped ? 2 * (h / per) * per + h % per : 2 * h, h2 = grouped ? h1 + per : h1 + 1;
-  const T* a1 = attn + (size_t)t * ld_a + (size_t)h1 * HD;
-  const T* a2 = attn + (size_t)t * ld_a + (size_t)h2 * HD;
+  const A* a1 = attn + (size_t)t * ld_a + (size_t)h1 * HD;
+  const A* a2 = attn + (size_t)t * ld_a + (size_t)h2 * HD;
   constexpr int kPerLane = 8;      // heads of up to 256 entries
   float val[kPerLane], ss = 0.f;
 #pragma unroll
@@ -361,17 +362,21 @@ LAB_EXPORT int lab_head_gate(void* out, int ld_o, const void* attn, int ld_a, co
   LAB_LAUNCH_CHECK();
 }
 
-// attn [tokens, ld_a] of T with 2 * H heads of HD entries; see map_difference_kernel for their order.
+// attn [tokens, ld_a] of T (attn_f32: of floats) with 2 * H heads of HD entries; see map_difference_kernel for their order.
 LAB_EXPORT int lab_map_difference(void* out, const void* attn, int ld_a, int tokens, int H, int V, int HD, int grouped,
-                                  int per, float lambda, float eps, float mult, int dtype, cudaStream_t stream) {
+                                  int per, float lambda, float eps, float mult, int attn_f32, int dtype,
+                                  cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (V > 256 || V > HD || H <= 0 || per < 1 || H % per) return (int)cudaErrorInvalidValue;
   const int blocks = (int)(((long long)tokens * H + kThreads / 32 - 1) / (kThreads / 32));
   if (dtype == LAB_F32)
-    lab_launch(map_difference_kernel<float>, dim3(blocks), dim3(kThreads), 0, stream, (float*)out, (const float*)attn, ld_a,
-               tokens, H, V, HD, grouped, per, lambda, eps, mult);
+    lab_launch(map_difference_kernel<float, float>, dim3(blocks), dim3(kThreads), 0, stream, (float*)out, (const float*)attn,
+               ld_a, tokens, H, V, HD, grouped, per, lambda, eps, mult);
+  else if (attn_f32)
+    lab_launch(map_difference_kernel<__nv_bfloat16, float>, dim3(blocks), dim3(kThreads), 0, stream, (__nv_bfloat16*)out,
+               (const float*)attn, ld_a, tokens, H, V, HD, grouped, per, lambda, eps, mult);
   else
-    lab_launch(map_difference_kernel<__nv_bfloat16>, dim3(blocks), dim3(kThreads), 0, stream, (__nv_bfloat16*)out,
+    lab_launch(map_difference_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(blocks), dim3(kThreads), 0, stream, (__nv_bfloat16*)out,
                (const __nv_bfloat16*)attn, ld_a, tokens, H, V, HD, grouped, per, lambda, eps, mult);
   LAB_LAUNCH_CHECK();
 }

@@ -316,28 +316,29 @@ def attention_plain(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tenso
                     row_pos: torch.Tensor, block_table: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
                     window: int, scale: float, out: torch.Tensor | None = None, keep_first: int = 0,
                     sink_one: bool = False, sink: torch.Tensor | None = None,
-                    dist_bias: torch.Tensor | None = None, softcap: float = 0.0) -> torch.Tensor:
+                    dist_bias: torch.Tensor | None = None, softcap: float = 0.0, out_f32: bool = False) -> torch.Tensor:
     """Attention of every row over its request's pages; q may be a column slice of the fused projection.
     `keep_first`: with a window, the first that many positions stay visible; `sink_one`: one more in the
     softmax's denominator; `sink` [n_q] 32-bit: exp(sink[h]) more instead; `dist_bias` [n_q, L] 32-bit: added to
     the scaled score by distance query - key, distances from L - 1 on sharing the last entry; `softcap` c > 0: the
-    scaled score s becomes c * tanh(s / c), before the bias."""
+    scaled score s becomes c * tanh(s / c), before the bias.  `out_f32`: the result is 32-bit, not rounded to q's type."""
     _on_gpu(q, cache_k, cache_v, row_req, row_pos, block_table, sink, dist_bias)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() >= n_q and sink.is_contiguous())
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.dim() == 2 and
                                  dist_bias.shape[0] == n_q and dist_bias.is_contiguous())
     tokens = q.shape[0]
     if out is None:
-        out = torch.empty((tokens, n_q * head_dim), dtype=q.dtype, device=q.device)
+        out = torch.empty((tokens, n_q * head_dim), dtype=torch.float32 if out_f32 else q.dtype, device=q.device)
     num_pages, kvh, page_size, d = cache_k.shape
     assert kvh == n_kv and d == head_dim and q.stride(1) == 1 and cache_k.dtype == q.dtype
+    assert out.dtype == (torch.float32 if out_f32 else q.dtype)
     assert block_table.dtype == torch.int32 and block_table.dim() == 2 and block_table.is_contiguous()
     _check(lib("attention_plain").lab_attention_plain(
         _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(cache_k), _ptr(cache_v), _ptr(row_req), _ptr(row_pos),
         _ptr(block_table), block_table.shape[1], tokens, n_q, n_kv, head_dim, page_size, num_pages, window,
         ctypes.c_float(scale), int(keep_first), int(bool(sink_one) or sink is not None), _ptr(sink), _ptr(dist_bias),
-        dist_bias.shape[1] if dist_bias is not None else 0, ctypes.c_float(softcap), dtype_code(q.dtype), _stream()),
-        "attention_plain")
+        dist_bias.shape[1] if dist_bias is not None else 0, ctypes.c_float(softcap), int(bool(out_f32)),
+        dtype_code(q.dtype), _stream()), "attention_plain")
     return out
 
 
@@ -741,7 +742,7 @@ TC05_BIAS_MAX = 4096     # entries of a distance table the tcgen05 prefill kerne
 
 def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requests, q_lens, max_kv_len,
                  n_q, n_kv, head_dim, window, scale, out=None, splits=None, scratch=None, keep_first=0, sink=None,
-                 dist_bias=None, softcap=0.0):
+                 dist_bias=None, softcap=0.0, out_f32=False):
     """Tensor-core attention: the prefill kernel serves requests with several new tokens,
     the split-KV decode kernel those with one.  A negative `window` means chunks of that many positions.
     `keep_first`: beside a window, the first that many positions stay visible.  `sink`: 32-bit numbers, one per
@@ -749,7 +750,7 @@ def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requ
     `dist_bias` [n_q, L] 32-bit: a number per head and distance query - key added to the scaled score, distances
     from L - 1 on sharing the last entry (the tcgen05 kernel keeps a head's table in shared memory, up to
     `TC05_BIAS_MAX` entries; longer tables run on the `mma.sync` prefill kernel).  `softcap` c > 0: the scaled score
-    s becomes c * tanh(s / c), before the bias."""
+    s becomes c * tanh(s / c), before the bias.  `out_f32`: the result is 32-bit, not rounded."""
     _on_gpu(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, sink, dist_bias)
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.dim() == 2 and
                                  dist_bias.shape[0] == n_q and dist_bias.is_contiguous())
@@ -760,9 +761,10 @@ def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requ
         raise KernelError(f"attention_tc: bfloat16 and a head size multiple of 16 up to 128, got {q.dtype}, {head_dim}")
     tokens = q.shape[0]
     if out is None:
-        out = torch.empty((tokens, n_q * head_dim), dtype=q.dtype, device=q.device)
+        out = torch.empty((tokens, n_q * head_dim), dtype=torch.float32 if out_f32 else q.dtype, device=q.device)
     num_pages, kvh, page_size, d = cache_k.shape
     assert kvh == n_kv and d == head_dim and q.stride(1) == 1 and q.stride(0) % 8 == 0
+    assert out.dtype == (torch.float32 if out_f32 else q.dtype)
     assert block_table.dim() == 2 and block_table.is_contiguous() and block_table.shape[0] >= n_requests
     L = lib("attention_tc", {"LAB_HEAD_DIM": head_dim})
     max_q = max(q_lens)
@@ -776,14 +778,14 @@ def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requ
             _ptr(out), out.stride(0), _ptr(q), q.stride(0), tokens, _ptr(cache_k), _ptr(cache_v), _ptr(q_start),
             _ptr(kv_len), _ptr(pos0), _ptr(block_table), block_table.shape[1], n_requests, max_q, n_q, n_kv,
             page_size, num_pages, window, ctypes.c_float(scale), 2, keep_first, _ptr(sink), _ptr(dist_bias), bias_len,
-            ctypes.c_float(softcap), _stream()),
+            ctypes.c_float(softcap), int(bool(out_f32)), _stream()),
             "attention_prefill_tc05")
     elif max_q > 1:
         _check(L.lab_attention_prefill(_ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(cache_k), _ptr(cache_v),
                                        _ptr(q_start), _ptr(kv_len), _ptr(pos0), _ptr(block_table),
                                        block_table.shape[1], n_requests, max_q, n_q, n_kv, page_size, num_pages,
                                        window, ctypes.c_float(scale), 2, _ptr(sink), keep_first, _ptr(dist_bias),
-                                       bias_len, ctypes.c_float(softcap), _stream()),
+                                       bias_len, ctypes.c_float(softcap), int(bool(out_f32)), _stream()),
                "attention_prefill")
     if n_decode:
         if splits is None:
@@ -801,14 +803,14 @@ def attention_tc(q, cache_k, cache_v, q_start, kv_len, pos0, block_table, n_requ
                                       _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.shape[1],
                                       n_requests, n_q, n_kv, page_size, num_pages, window, ctypes.c_float(scale),
                                       splits, _ptr(scratch), 1 if in_cluster else 0, keep_first, _ptr(sink),
-                                      _ptr(dist_bias), bias_len, ctypes.c_float(softcap), _stream()),
+                                      _ptr(dist_bias), bias_len, ctypes.c_float(softcap), int(bool(out_f32)), _stream()),
                "attention_decode",
                2 if splits > 1 and not in_cluster else 1)
     return out
 
 
 def attention(q, cache_k, cache_v, ctx, group, n_q, n_kv, head_dim, window, scale, chunk=0, keep_first=0,
-              sink_one=False, sink=None, dist_bias=None, softcap=0.0):
+              sink_one=False, sink=None, dist_bias=None, softcap=0.0, out_f32=False):
     """Causal attention of every row over its request's cached keys: all of them, the last `window`, or
     (with `chunk`) those of the row's own chunk of `chunk` positions, chunks counted from position 0.  The
     kernels take the mask as one number: a window as it is, a chunk as its negative.  `keep_first`: beside a
@@ -816,7 +818,7 @@ def attention(q, cache_k, cache_v, ctx, group, n_q, n_kv, head_dim, window, scal
     holds one more (a key with score 0 and no value); `sink` [n_q] 32-bit: it holds exp(sink[h]) more instead (a
     learned score of that key, unscaled); `dist_bias` [n_q, L] 32-bit: a number per head and distance query - key
     added to the scaled score, distances from L - 1 on sharing the last entry; `softcap` c > 0: the scaled score s
-    becomes c * tanh(s / c), before the bias."""
+    becomes c * tanh(s / c), before the bias; `out_f32`: the result is 32-bit, not rounded to q's type."""
     if sink is not None:
         sink_one = False
     if chunk:
@@ -829,11 +831,11 @@ def attention(q, cache_k, cache_v, ctx, group, n_q, n_kv, head_dim, window, scal
         # the denominator's extra one is a sink of 0 for every head
         return attention_tc(q, cache_k, cache_v, ctx.q_start, ctx.kv_len, ctx.pos0, group.block_table,
                             ctx.n_requests, ctx.q_lens, ctx.max_kv_len, n_q, n_kv, head_dim, window, scale,
-                            keep_first=keep_first, dist_bias=dist_bias, softcap=softcap,
+                            keep_first=keep_first, dist_bias=dist_bias, softcap=softcap, out_f32=out_f32,
                             sink=sink if sink is not None else (_zero_sinks(q.device, n_q) if sink_one else None))
     return attention_plain(q, cache_k, cache_v, ctx.row_req, ctx.row_pos, group.block_table, n_q, n_kv, head_dim,
                            window, scale, keep_first=keep_first, sink_one=sink_one, sink=sink, dist_bias=dist_bias,
-                           softcap=softcap)
+                           softcap=softcap, out_f32=out_f32)
 
 
 _zero_sink_cache: dict = {}
@@ -1278,7 +1280,7 @@ def latent_attention_plain_form(q: torch.Tensor, cache: torch.Tensor, w_up: torc
                                     _ptr(ctx.q_start), _ptr(ctx.kv_len), _ptr(ctx.pos0), _ptr(table), table.shape[1],
                                     ctx.n_requests, ctx.max_q_len, heads, heads, page_size, num_pages, window,
                                     ctypes.c_float(scale), int(at_least), _ptr(sink), 0, None, 0,
-                                    ctypes.c_float(0.0), _stream()), "attention_prefill")
+                                    ctypes.c_float(0.0), 0, _stream()), "attention_prefill")
     return out
 
 
@@ -1450,18 +1452,21 @@ def head_gate(attn: torch.Tensor, proj: torch.Tensor, gate_at: int, per_head: bo
 
 
 def map_difference(attn: torch.Tensor, heads: int, vdim: int, head: int, lam: float, eps: float, mult: float,
-                   group: int = 0) -> torch.Tensor:
+                   group: int = 0, dtype: torch.dtype | None = None) -> torch.Tensor:
     """Two score maps' outputs combined per head: a1 - lam * a2 over its root mean square within the head's `vdim`
-    entries (eps inside the root), times `mult`, packed [tokens, heads * vdim] in the storage type of `attn`
-    [tokens, 2 * heads * head].  A head's maps are heads 2h and 2h + 1 of `attn`; `group` > 0 (heads of a group): the
+    entries (eps inside the root), times `mult`, packed [tokens, heads * vdim] in `dtype` (None: that of `attn`);
+    `attn` [tokens, 2 * heads * head] in the same type or in 32-bit.  A head's maps are heads 2h and 2h + 1 of `attn`; `group` > 0 (heads of a group): the
     queries are ordered by group, map and head within the group."""
     _on_gpu(attn)
     tokens = attn.shape[0]
     assert attn.stride(1) == 1 and attn.shape[1] == 2 * heads * head and vdim <= head
-    out = torch.empty((tokens, heads * vdim), dtype=attn.dtype, device=attn.device)
+    dtype = dtype or attn.dtype
+    assert attn.dtype in (dtype, torch.float32)
+    out = torch.empty((tokens, heads * vdim), dtype=dtype, device=attn.device)
     _check(lib("norm_attention").lab_map_difference(
         _ptr(out), _ptr(attn), attn.stride(0), tokens, heads, vdim, head, int(group > 0), max(int(group), 1),
-        ctypes.c_float(lam), ctypes.c_float(eps), ctypes.c_float(mult), dtype_code(attn.dtype), _stream()), "map_difference")
+        ctypes.c_float(lam), ctypes.c_float(eps), ctypes.c_float(mult), int(attn.dtype == torch.float32), dtype_code(dtype),
+        _stream()), "map_difference")
     return out
 
 

@@ -24,7 +24,8 @@ class DifferentialAttention(Mixer):
     with the whole key meets that half alone; where values are twice as wide as keys nothing is padded.  Split form,
     for heads whose two keys together are too wide for the tensor-core kernels: every map is a key/value head of its
     own, with the values stored twice; the queries are then ordered by group, map and head within the group (the
-    rows of W_q are reordered at load time).  One kernel norms, rounds and stores; one combines the maps."""
+    rows of W_q are reordered at load time).  One kernel norms, rounds and stores; one combines the maps, whose outputs
+    leave the attention kernels in 32-bit: the difference of two alike maps is small next to their own rounding."""
     decode_graph_safe = True
 
     @classmethod
@@ -93,9 +94,9 @@ class DifferentialAttention(Mixer):
                                 self.dtype, norm_eps=self.eps, q_norm_w=self.norm_q, k_norm_w=self.norm_k,
                                 maps=2 if self.packed else 1, v_rep=1 if self.packed else 2)
         attn = ops.attention(q, cache.k, cache.v, ctx, group, 2 * self.heads, n_kv, self.head, self.window, self.scale,
-                             softcap=self.softcap)
+                             softcap=self.softcap, out_f32=True)
         y = ops.map_difference(attn, self.heads, self.vdim, self.head, self.lam, self.eps, 1.0 - self.diff,
-                               group=0 if self.packed else self.per)
+                               group=0 if self.packed else self.per, dtype=self.dtype)
         return ops.linear(y, self.w_o, None, out_f32=True, allow_partial=True)
 
 

@@ -380,7 +380,10 @@ def test_window_and_cap_in_every_attention_kernel(D, H, G, page, window, cap):
             keys.append(_np(k)), vals.append(_np(v))
             _fill_pages(ck, cv, table, r, k, v, page)
         q = _t(rng.standard_normal((sum(q_lens), H * D)), dtype)
-        got = _np(ops.attention(q, ck, cv, ctx, ctx.groups[0], H, G, D, window, scale, softcap=cap))
+        wide = ops.attention(q, ck, cv, ctx, ctx.groups[0], H, G, D, window, scale, softcap=cap, out_f32=True)
+        rounded = ops.attention(q, ck, cv, ctx, ctx.groups[0], H, G, D, window, scale, softcap=cap)
+        assert wide.dtype == torch.float32 and rounded.dtype == dtype and torch.equal(wide.to(dtype), rounded)
+        got = _np(wide)
         at = far = 0
         for r, (n, p0) in enumerate(zip(q_lens, pos0)):
             rows = _np(q[at: at + n]).reshape(n, H, D)
@@ -459,6 +462,13 @@ def test_difference_of_two_maps(H, V, head, group):
         x = _np(_t(a, dtype))[..., :V]
         want = pn.two_map_difference(x[:, :, 0], x[:, :, 1], 0.8, 1e-3, 0.45)
         assert np.abs(got - want).max() < (1e-5 if dtype == torch.float32 else 0.02)
+        # two maps that differ by less than their rounding to bfloat16, a weight near one: 32-bit maps keep the difference
+        close = np.repeat(a[:, :, :1], 2, axis=2) * np.array([1.0, 1.001])[:, None]
+        flat = close.reshape(9, -1) if not group else close.reshape(9, H // group, group, 2, head).transpose(0, 1, 3, 2, 4).reshape(9, -1)
+        out = ops.map_difference(_t(flat), H, V, head, 1.0, 1e-12, 0.55, group=group, dtype=dtype)
+        x = _np(_t(close))[..., :V]
+        want = pn.two_map_difference(x[:, :, 0], x[:, :, 1], 1.0, 1e-12, 0.45)
+        assert out.dtype == dtype and np.abs(_np(out).reshape(9, H, V) - want).max() < (1e-2 if V > 1 else 2.0)
 
 
 @pytest.mark.parametrize("mixer", [attention(4, 2, 16, 24, window=9, softcap=3.0, diff=0.4, scale=0.7),
