@@ -27,6 +27,8 @@ constexpr int PF_BM = 64, PF_BN = 64, PF_THREADS = 128;
 constexpr int PF_TILE_BYTES = PF_BN * ROW_BYTES;
 constexpr int PF_SMEM = PF_BM * ROW_BYTES + 4 * PF_TILE_BYTES;  // Q + 2 stages of (K, V)
 
+// MORE: a build of its own for the soft cap and the 32-bit output, which the others then cost nothing.
+template <bool MORE>
 __global__ void __launch_bounds__(PF_THREADS) attention_prefill_kernel(
     void* __restrict__ out, int out_stride, const __nv_bfloat16* __restrict__ q, int q_stride,
     const __nv_bfloat16* __restrict__ cache_k, const __nv_bfloat16* __restrict__ cache_v,
@@ -35,6 +37,7 @@ __global__ void __launch_bounds__(PF_THREADS) attention_prefill_kernel(
     float scale_log2, int min_q_len, const float* __restrict__ sink, int keep, const float* __restrict__ dist_bias,
     int bias_len, float cap_log2, float arg_log2, int out_f32) {
   extern __shared__ __align__(16) uint8_t smem[];
+  if constexpr (!MORE) cap_log2 = 0.f, out_f32 = 0;
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.z, h = blockIdx.y;
@@ -190,7 +193,8 @@ struct DcLayout {
 // elements: each split stores the (acc, max, sum) of those elements straight into the shared
 // memory of the CTA that merges them (remote stores do not stall, remote loads would), and after
 // one cluster barrier everyone finds all it needs at home: no scratch and no merge kernel.
-template <bool CLUSTER = false>
+// MORE: as in the prefill kernel.
+template <bool CLUSTER, bool MORE>
 __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
     void* __restrict__ out, int out_stride, const __nv_bfloat16* __restrict__ q, int q_stride,
     __nv_bfloat16* __restrict__ cache_k, __nv_bfloat16* __restrict__ cache_v,
@@ -199,6 +203,7 @@ __global__ void __launch_bounds__(DC_THREADS) attention_decode_kernel(
     float* __restrict__ part_acc, float* __restrict__ part_ml, int keep, const float* __restrict__ sink,
     const float* __restrict__ dist_bias, int bias_len, float cap_log2, float arg_log2, int out_f32) {
   extern __shared__ __align__(16) uint8_t smem[];
+  if constexpr (!MORE) cap_log2 = 0.f, out_f32 = 0;
   using L = DcLayout<CLUSTER>;
   pdl_trigger();
   // Until pdl_wait() below only what no kernel of this step writes is read: the step's metadata
@@ -471,14 +476,16 @@ LAB_EXPORT int lab_attention_prefill(void* out, int out_stride, const void* q, i
                                      float softcap, int out_f32, cudaStream_t stream) {
   if (requests <= 0 || max_q_len <= 0) return 0;
   if (n_q % n_kv || q_stride % 8 || (((uintptr_t)q) & 15)) return (int)cudaErrorInvalidValue;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
+  const bool more = softcap > 0.f || out_f32;
+  auto kernel = more ? attention_prefill_kernel<true> : attention_prefill_kernel<false>;
+  static bool configured[2] = {};
+  if (!configured[more]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
     if (e != cudaSuccess) return (int)e;
-    configured = true;
+    configured[more] = true;
   }
   dim3 grid((max_q_len + PF_BM - 1) / PF_BM, n_q, requests);
-  return (int)lab_launch(attention_prefill_kernel, grid, dim3(PF_THREADS), (size_t)PF_SMEM, stream,
+  return (int)lab_launch(kernel, grid, dim3(PF_THREADS), (size_t)PF_SMEM, stream,
                          out, out_stride, (const __nv_bfloat16*)q, q_stride,
                          (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v, q_start, kv_len, pos0,
                          block_table, max_blocks, n_q, n_kv, page_size, num_pages, window, scale * LOG2E, min_q_len,
@@ -502,15 +509,16 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
   int device = 0;
   if (cudaGetDevice(&device) != cudaSuccess || device < 0 || device >= 64) return (int)cudaErrorInvalidDevice;
   if (!configured[device]) {
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         DcLayout<false>::SMEM);
-    if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(attention_decode_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                               DcLayout<true>::SMEM);
+    cudaError_t e = cudaSuccess;
+    for (auto k : {attention_decode_kernel<false, false>, attention_decode_kernel<false, true>})
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, DcLayout<false>::SMEM);
+    for (auto k : {attention_decode_kernel<true, false>, attention_decode_kernel<true, true>})
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, DcLayout<true>::SMEM);
     if (e != cudaSuccess) return (int)e;
     configured[device] = true;
   }
   const int group = n_q / n_kv, m_tiles = (group + 15) / 16;
+  const bool more = softcap > 0.f || out_f32;
   dim3 grid(splits, n_kv * m_tiles, requests);
   if (cluster) {
     cudaLaunchConfig_t cfg = {};
@@ -527,7 +535,8 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = g_lab_pdl ? 2 : 1;
-    return (int)cudaLaunchKernelEx(&cfg, attention_decode_kernel<true>, out, out_stride,
+    return (int)cudaLaunchKernelEx(&cfg, more ? attention_decode_kernel<true, true> : attention_decode_kernel<true, false>,
+                                   out, out_stride,
                                    (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v,
                                    q_start, kv_len, block_table, max_blocks, n_q, n_kv, page_size, num_pages, window,
                                    scale * LOG2E, splits, (float*)nullptr, (float*)nullptr, keep, sink, dist_bias,
@@ -535,7 +544,7 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
   }
   float* part_acc = scratch;
   float* part_ml = scratch ? scratch + (size_t)requests * n_q * splits * D : nullptr;
-  cudaError_t e = lab_launch(attention_decode_kernel<false>, grid, dim3(DC_THREADS), (size_t)DcLayout<false>::SMEM, stream,
+  cudaError_t e = lab_launch(more ? attention_decode_kernel<false, true> : attention_decode_kernel<false, false>, grid, dim3(DC_THREADS), (size_t)DcLayout<false>::SMEM, stream,
                              out, out_stride, (const __nv_bfloat16*)q, q_stride,
                              (__nv_bfloat16*)cache_k, (__nv_bfloat16*)cache_v, q_start, kv_len, block_table,
                              max_blocks, n_q, n_kv, page_size, num_pages, window, scale * LOG2E, splits, part_acc,

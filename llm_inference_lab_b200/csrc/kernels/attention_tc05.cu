@@ -80,6 +80,8 @@ struct Barriers {
   int abort_flag;
 };
 
+// MORE: a build of its own for the soft cap and the 32-bit output, which the others then cost nothing.
+template <bool MORE>
 __global__ void __launch_bounds__(THREADS) attention_prefill_tc05_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, void* __restrict__ out, int out_stride,
@@ -88,6 +90,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc05_kernel(
     const int* __restrict__ block_table, int max_blocks, int n_q, int n_kv, int page_size, int num_pages, int window,
     float scale_log2, int min_q_len, int keep, const float* __restrict__ sink, const float* __restrict__ dist_bias,
     int bias_len, float bias_mult, float cap_log2, float arg_log2, int out_f32) {
+  if constexpr (!MORE) cap_log2 = 0.f, out_f32 = 0;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   Barriers* bar = reinterpret_cast<Barriers*>(smem + OFF_BAR);
@@ -493,15 +496,16 @@ LAB_EXPORT int lab_attention_prefill_tc05(void* out, int out_stride, const void*
   const long long cache_rows = (long long)num_pages * n_kv * page_size;
   if ((rc = lab_make_map_bf16(&mk, cache_k, cache_rows, D, D, page_size))) return rc;
   if ((rc = lab_make_map_bf16(&mv, cache_v, cache_rows, D, D, page_size))) return rc;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e =
-        cudaFuncSetAttribute(attention_prefill_tc05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+  const bool more = softcap > 0.f || out_f32;
+  auto kernel = more ? attention_prefill_tc05_kernel<true> : attention_prefill_tc05_kernel<false>;
+  static bool configured[2] = {};
+  if (!configured[more]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return (int)e;
-    configured = true;
+    configured[more] = true;
   }
   dim3 grid(n_q, (max_q_len + BM - 1) / BM, requests);
-  return (int)lab_launch(attention_prefill_tc05_kernel, grid, dim3(THREADS), (size_t)SMEM, stream, mq, mk, mv,
+  return (int)lab_launch(kernel, grid, dim3(THREADS), (size_t)SMEM, stream, mq, mk, mv,
                          out, out_stride, (const __nv_bfloat16*)cache_k, (const __nv_bfloat16*)cache_v,
                          q_start, kv_len, pos0, block_table, max_blocks, n_q, n_kv, page_size, num_pages, window,
                          softcap > 0.f ? 1.f : scale * LOG2E, min_q_len, window > 0 && keep_first > 0 ? keep_first : 0, sink,
